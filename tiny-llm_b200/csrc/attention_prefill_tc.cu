@@ -74,8 +74,8 @@ __host__ __device__ constexpr uint32_t tc_instr_desc(int n, bool b_mn) {
            | (static_cast<uint32_t>(TC_BM >> 4) << 24);
 }
 
-// ex2.approx.ftz: one MUFU instruction (exp2f() adds denormal-range scaling, ~3 more instructions per element; ncu of the
-// first version: 10.7 instructions per score element, issue slots 54 % busy with the tensor pipe at 40 %).  Relative error
+// ex2.approx.ftz: the hardware approximation without the denormal range that exp2f() keeps (ncu of the first version: issue
+// slots 54 % busy with the tensor pipe at 40 %).  Relative error
 // 2^-22; the reference kernel uses fast::exp2 (paged_attention.metal:428-436).
 __device__ __forceinline__ float tc_ex2(float x) {
     float y;
@@ -205,8 +205,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
         // on the next tile's scores while the softmax warps are busy with this tile's.
         // The whole warp walks the loop (uniform control flow, running stage / phase counters, descriptors derived by
         // adding to three base descriptors), one elected lane issues (tc05.cuh: g_elect_one - behind `if (lane == 0)`
-        // every tcgen05 instruction sat in an ELECT loop with its operands moved through R2UR, and the issue latency
-        // of a tile was of the order of its 512 cycles of tensor work).
+        // the issue latency of a tile, by the cycle trace, was of the order of its 512 cycles of tensor work).
         if (n_tiles > 0) {
             constexpr uint32_t idesc_s = tc_instr_desc(TC_BN, false);
             constexpr uint32_t idesc_o = tc_instr_desc(TC_D, true);

@@ -167,9 +167,8 @@ __global__ void __launch_bounds__(G_THREADS, 1) w4a16_gemm_kernel(const __grid_c
     } else if (warp == 1) {
         // ------------------------------------------------ MMA issuer
         // The whole warp walks the loop (uniform control flow, running stage / phase counters instead of a division per
-        // block), one elected lane issues: behind `if (lane == 0)` the compiler wrapped every tcgen05 instruction in an
-        // ELECT loop and moved its operands through R2UR - ~1000 cycles of issue latency per reduction block, more than
-        // the 512 cycles of tensor work of a two-tile stage (tc05.cuh: g_elect_one).
+        // block), one elected lane issues: behind `if (lane == 0)` the cycle trace showed ~1000 cycles of issue latency per
+        // reduction block, more than the 512 cycles of tensor work of a two-tile stage (tc05.cuh: g_elect_one).
         constexpr uint32_t idesc = g_instr_desc<T>();
         const uint64_t adesc0 = g_smem_desc(a_base), bdesc0 = g_smem_desc(b_base);
         int s = 0;

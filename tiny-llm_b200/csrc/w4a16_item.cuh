@@ -2,12 +2,12 @@
 // the register-pipelined weight unit and the tensor-core consumer.
 //
 // Why this shape (measured on B200, profiles/r01_kbench_*): the first three streaming kernels
-// all stalled at ~2 TB/s no matter how the bytes were fetched.  SASS of the cp.async-ring
-// version showed 334 instructions per 1-KiB weight group per warp - the kernel was
-// instruction-issue bound, not memory bound.  The budget below is ~100 per KiB:
+// all stalled at ~2 TB/s no matter how the bytes were fetched: the profiler's executed-instruction
+// count per byte of weights made the cp.async-ring version instruction-issue bound, not memory
+// bound.  The form below does less work per weight:
 //
 //   * weights go global -> registers (ld.global.nc, 128-bit, immediate offsets from one running
-//     pointer per row); no shared-memory ring, so no LDGSTS, no wait_group/syncwarp, no slot math;
+//     pointer per row); no shared-memory ring, so no cp.async, no wait_group/syncwarp, no slot math;
 //   * a lane turns four codes into two exact bf16 (128+q) pairs with ONE lop3 each (mask in the
 //     constant bank, magic in a register) plus a shift for three of the four nibble positions;
 //   * the B fragments of a unit are four 128-bit shared loads at compile-time offsets from one
@@ -24,10 +24,9 @@
 
 namespace tl {
 
-// Opaque to ptxas (constant memory may be rewritten by the host), which keeps (x & mask) | magic
-// a single LOP3 with the mask read from the constant bank.
+// In constant memory, so that (x & mask) | magic takes its mask from there instead of from a register.
 static __constant__ uint32_t k_w4_mask = 0x000F000Fu;
-// Experiment switch: x >> s as the high word of x * 2^(32-s) (IMAD.HI, FMA pipe) instead of SHF
+// Experiment switch: x >> s as the high word of x * 2^(32-s) (a multiply) instead of a shift
 // (ALU pipe).  Measured slower on B200 (lm_head 56 -> 69 us): kept only for the record.
 #ifndef W4_SHR_IMADHI
 #define W4_SHR_IMADHI 0

@@ -34,12 +34,11 @@ int launch_w4a16_stream(const void *scales, const void *biases, const void *a, c
 
 // ---------------------------------------------------------------------------
 // v5: register-pipelined streaming, contiguous rows per CTA (see w4a16_item.cuh for the
-// instruction budget of the inner loop).
+// inner loop).
 //
 // History, all measured on B200 (profiles/r01_kbench_*, tools/s4_timeline.py):
 //   v1 (register prefetch, 2 KB in flight per warp), v2 (producer warp + 256-byte cp.async.bulk
-//   ring) and v3 (per-warp cp.async rings) stalled near 2 TB/s: ~330 instructions per KiB of
-//   weights - issue bound.  v4 (register pipeline, ~120 instructions per KiB) reached 3.9 TB/s on
+//   ring) and v3 (per-warp cp.async rings) stalled near 2 TB/s: issue bound.  v4 (register pipeline) reached 3.9 TB/s on
 //   the tied head but dealt 16-row tiles to fixed-size warp teams: 1216 tiles over 1184 teams
 //   made 32 teams work twice as long as the rest (gate|up: 11 us instead of 6), and every tile
 //   ended with two named barriers and a dependent residual load.

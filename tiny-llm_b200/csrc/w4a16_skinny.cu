@@ -26,7 +26,7 @@
 // 64-wide block with the tile in shared memory 156 us -> two alternating groups, thread = row 143 us -> tile in tensor
 // memory (6 stages instead of 2) 136 us -> MMA warp on elect.sync 112 us -> 128-wide blocks (one barrier round trip per
 // quantisation group) 94 us (36.5 % of the HBM rate; 16 rows: 79 us, 41 %).  The per-block cycle trace (tools/skinny_blocks.py) showed each time which actor the
-// others were waiting for; the arithmetic of the dequantisers (~2.9 instructions per weight) is the floor.
+// others were waiting for; the arithmetic of the dequantisers is the floor.
 #include <stdlib.h>
 
 #include <mutex>
