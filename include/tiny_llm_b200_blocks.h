@@ -41,10 +41,20 @@ int tlb_embed_rows(const int32_t *ids, const void *table, float *x32, void *h, i
 int tlb_norm_residual(const void *y, int y_is_f32, const void *w, float weight_offset, const void *scale, float eps, float *residual,
                       void *h, int rows, int dim, int dtype, void *stream);
 
+/* The same start of the residual stream with a scale, a second table and the norms that read it first:
+ *   x32[t] = table[ids[t]] * scale (+ pairs[r] if pairs != NULL), pairs [buckets + 1, dim],
+ *   r = (id before t in its sequence * mul_prev + ids[t] * mul_cur) mod buckets, r = buckets for tok_pos[t] == 0;
+ * the token before is ids[t - 1] when tok_seq[t - 1] == tok_seq[t], else seq_prev[tok_seq[t]].  mul_prev, mul_cur in
+ * [0, buckets).  h1 (h2), if not NULL: x32 / rms(x32) * w1 (w2) rounded to `dtype`. */
+int tlb_embed_pairs(const int32_t *ids, const int32_t *tok_pos, const int32_t *tok_seq, const int32_t *seq_prev, const void *table, int vocab, float scale,
+                    const void *pairs, long long buckets, long long mul_prev, long long mul_cur, float *x32, const void *w1, void *h1, const void *w2,
+                    void *h2, float eps, int tokens, int dim, int dtype, void *stream);
+
 /* End of a sublayer, fused with the next norm: residual += a (+ b, if b != NULL) in fp32, then, if w != NULL,
- * h = residual / rms(residual) * w rounded to `dtype`.  a_row != 0: `a` is one row [dim] added to every row. */
-int tlb_add_norm(float *residual, const float *a, int a_row, const float *b, const void *w, float eps, void *h, int rows, int dim, int dtype,
-                 void *stream);
+ * h = residual / rms(residual) * w rounded to `dtype`, and, if w2 != NULL, h2 = residual / rms(residual) * w2 (two sublayers
+ * that read the stream side by side).  a_row != 0: `a` is one row [dim] added to every row. */
+int tlb_add_norm(float *residual, const float *a, int a_row, const float *b, const void *w, float eps, void *h, const void *w2, void *h2, int rows,
+                 int dim, int dtype, void *stream);
 
 /* y = coef * (a / rms(a) * wa + b / rms(b) * wb); a, b, y fp32 [rows, dim], wa, wb `dtype` [dim]. */
 int tlb_norm_mix2(const float *a, const void *wa, const float *b, const void *wb, float coef, float eps, float *y, int rows, int dim, int dtype,
@@ -56,8 +66,11 @@ int tlb_norm_mix2(const float *a, const void *wa, const float *b, const void *wb
 int tlb_rope_rows(void *x, long long row_stride, long long head_stride, int first, int heads, int dims, int interleaved, double base,
                   double factor, const int32_t *tok_pos, int rows, int dtype, void *stream);
 /* The same angles as fp32 tables cos_out, sin_out [rows, dims / 2], for kernels that rotate in fp32 on their way into a
- * recurrence (tlb_decay_scan). */
-int tlb_rope_table(const int32_t *tok_pos, int rows, int dims, double base, double factor, float *cos_out, float *sin_out, void *stream);
+ * recurrence (tlb_decay_scan) or into the cache (tlb_qk_whole_prepare).  ramp_factor != 1: frequency f_i becomes
+ * f_i / ramp_factor * r + f_i * (1 - r), r = clamp((i - ramp_lo) / max(ramp_hi - ramp_lo, 0.001), 0, 1) (low frequencies
+ * stretched, high ones kept); gain multiplies both tables. */
+int tlb_rope_table(const int32_t *tok_pos, int rows, int dims, double base, double factor, double ramp_factor, double ramp_lo, double ramp_hi, double gain,
+                   float *cos_out, float *sin_out, void *stream);
 
 /* Latent cache append: for every token, the first `rank` entries of down[t,:] are RMS-normed (plain weight) and the last
  * `rot` entries rotated by the token's position; both are stored at the token's slot of slab [pages, page_size, rank+rot]
@@ -105,14 +118,14 @@ size_t tlb_latent_attention_mma_workspace(int num_tiles, int heads, int rank, in
 
 /* Grouped-query softmax attention over a paged cache whose row (one token) is [kv_heads * dk keys | kv_heads * dv values].
  * q [T, heads, dk] and out [T, heads, dv] are views with token / head strides in elements.  Token t sees key j <= tok_pos[t]
- * and, mask 1: tok_pos[t] - j < mask_size (sliding window); mask 2: j / mask_size == tok_pos[t] / mask_size (chunks counted
+ * and, mask 1: tok_pos[t] - j < mask_size (sliding window) or j < keep_first (kept first positions; 0 = none); mask 2: j / mask_size == tok_pos[t] / mask_size (chunks counted
  * from position 0); mask 0: all.  score = scale * q.k, then softcap * tanh(score / softcap) when softcap > 0; sink != 0 adds
  * exp(0) to the softmax's denominator; gate != NULL multiplies head h's output by sigmoid(gate[t * g_token + h]).
  * tiles [num_tiles, 3] as for latent attention, cut to at most tlb_paged_attention_tile_tokens(heads, kv_heads) tokens. */
 int tlb_paged_attention_tile_tokens(int heads, int kv_heads);
 int tlb_paged_attention(const void *q, long long q_token, long long q_head, const void *slab, int num_pages, int page_size, int dk, int dv,
                         int heads, int kv_heads, const int32_t *block_table, int max_pages, const int32_t *tiles, int num_tiles,
-                        const int32_t *tok_pos, int mask, int mask_size, float scale, float softcap, int sink, const void *gate,
+                        const int32_t *tok_pos, int mask, int mask_size, int keep_first, float scale, float softcap, int sink, const void *gate,
                         long long g_token, void *out, long long o_token, long long o_head, const float *head_bias, int weights, int dtype,
                         void *stream);
 /* head_bias [heads] fp32 (or NULL): with sink != 0 the sink's term is exp(head_bias[h]) instead of exp(0).  weights 1: no
@@ -124,7 +137,7 @@ int tlb_paged_attention_mma_tile_tokens(int heads, int kv_heads);
 int tlb_paged_attention_mma_supported(int dk, int dv, int kv_heads, int page_size);
 int tlb_paged_attention_mma(const void *q, long long q_token, long long q_head, const void *slab, int num_pages, int page_size, int dk, int dv,
                             int heads, int kv_heads, const int32_t *block_table, int max_pages, const int32_t *tiles, int num_tiles,
-                            const int32_t *tok_pos, int mask, int mask_size, float scale, float softcap, int sink, const void *gate,
+                            const int32_t *tok_pos, int mask, int mask_size, int keep_first, float scale, float softcap, int sink, const void *gate,
                             long long g_token, void *out, long long o_token, long long o_head, int splits, void *workspace,
                             size_t workspace_bytes, const float *head_bias, int weights, void *stream);
 /* splits > 1 cuts every tile's key range over that many CTAs (few query rows, long key ranges) and a second launch merges the
@@ -213,8 +226,8 @@ int tlb_softcap_rows(float *x, int rows, int width, float cap, void *stream);
 /* dst[r, 0:dim] = src[r, :] rounded to `dtype`; dst rows dst_stride elements apart. */
 int tlb_cast_rows(const float *src, void *dst, long long dst_stride, int rows, int dim, int dtype, void *stream);
 
-/* out[t, j] = act(gu[t, j]) * gu[t, width + j]; act 0 = silu, 1 = gelu (tanh form). */
-int tlb_gated_act(const void *gu, void *out, int rows, int width, int act, float limit, float slope, int dtype, void *stream);
+/* out[t, j] = act(gu[t, j]) * gu[t, width + j]; act 0 = silu, 1 = gelu (tanh form).  out rows are out_row elements apart. */
+int tlb_gated_act(const void *gu, void *out, long long out_row, int rows, int width, int act, float limit, float slope, int dtype, void *stream);
 /* act 3: g = min(gate, limit), u = clamp(up, -limit, limit), out = g sigmoid(slope g) (u + 1). */
 
 /* n residual streams xs [rows, n, dim] fp32 around a sublayer, n <= 8.  With write_w (mix [n, n] indexed [from, to], then

@@ -410,17 +410,20 @@ short_conv_kernel(const T *__restrict__ x, long long x_token, const T *__restric
 }
 
 // cos / sin of position * base^(-2 i / dims) / factor for every token: tables [rows, dims / 2] fp32 that kernels rotating in
-// fp32 (those that feed a recurrence) read instead of evaluating the angle themselves.
-__global__ void rope_table_kernel(const int32_t *__restrict__ tok_pos, int dims, double log2_base, double inv_factor, float *__restrict__ cs,
-                                  float *__restrict__ sn) {
+// fp32 (those that feed a recurrence, or the cache) read instead of evaluating the angle themselves.  The ramp divides the low
+// frequencies by a factor of their own and leaves the high ones, linear in the pair's number in between; gain scales both tables.
+__global__ void rope_table_kernel(const int32_t *__restrict__ tok_pos, int dims, double log2_base, double inv_factor, double inv_ramp_factor, double ramp_lo,
+                                  double ramp_hi, double gain, float *__restrict__ cs, float *__restrict__ sn) {
     const int row = blockIdx.x, half = dims / 2;
     const int pos = tok_pos[row];
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
         double freq = exp2(-2.0 * (double)i / (double)dims * log2_base) * inv_factor;
+        double ramp = fmin(fmax(((double)i - ramp_lo) / fmax(ramp_hi - ramp_lo, 0.001), 0.0), 1.0);
+        freq = freq * inv_ramp_factor * ramp + freq * (1.0 - ramp);
         double s, c;
         sincos((double)pos * freq, &s, &c);
-        cs[(size_t)row * half + i] = (float)c;
-        sn[(size_t)row * half + i] = (float)s;
+        cs[(size_t)row * half + i] = (float)(c * gain);
+        sn[(size_t)row * half + i] = (float)(s * gain);
     }
 }
 
@@ -530,10 +533,12 @@ int tlb_short_conv(const void *x, long long x_token, const void *taps, const voi
     return TL_OK;
 }
 
-int tlb_rope_table(const int32_t *tok_pos, int rows, int dims, double base, double factor, float *cos_out, float *sin_out, void *stream) {
+int tlb_rope_table(const int32_t *tok_pos, int rows, int dims, double base, double factor, double ramp_factor, double ramp_lo, double ramp_hi, double gain,
+                   float *cos_out, float *sin_out, void *stream) {
     if (rows <= 0 || dims <= 0) return TL_OK;
-    if (!tok_pos || !cos_out || !sin_out || (dims & 1) || base <= 0 || !(factor > 0)) return tl::fail(TL_EINVAL, "rope_table: bad argument");
-    rope_table_kernel<<<rows, 64, 0, as_stream(stream)>>>(tok_pos, dims, log2(base), 1.0 / factor, cos_out, sin_out);
+    if (!tok_pos || !cos_out || !sin_out || (dims & 1) || base <= 0 || !(factor > 0) || !(ramp_factor > 0))
+        return tl::fail(TL_EINVAL, "rope_table: bad argument");
+    rope_table_kernel<<<rows, 64, 0, as_stream(stream)>>>(tok_pos, dims, log2(base), 1.0 / factor, 1.0 / ramp_factor, ramp_lo, ramp_hi, gain, cos_out, sin_out);
     TL_LAUNCH_CHECK("rope_table");
     return TL_OK;
 }

@@ -5,7 +5,8 @@
 // consecutive tokens of one sequence x up to 4 query heads of ONE key/value head (16 query rows) and streams each
 // 32-key tile of that head through shared memory once for all of them.  What a position may see is a parameter:
 //   mask 0  every earlier position (causal)
-//   mask 1  itself and the size-1 positions before it (sliding window)
+//   mask 1  itself and the size-1 positions before it (sliding window), and with keep_first > 0 also the sequence's first
+//           keep_first positions, however far back they are: their key tiles come ahead of the window's
 //   mask 2  the earlier positions of its own block of `size` positions, blocks counted from position 0 (chunks)
 // and so are a tanh soft cap on the scaled scores, a sink (one more term in the softmax's denominator that carries no
 // value: exp(0), or exp(head_bias[h]) with a learned number per head) and a per-head output gate (the output of head h
@@ -25,9 +26,9 @@ constexpr int kPaHeads = 4;   // most query heads of one group per CTA
 
 __host__ __device__ inline int pa_heads_per_cta(int group) { return group < kPaHeads ? group : kPaHeads; }
 
-__device__ __forceinline__ bool pa_visible(int p, int key, int mask, int size) {
+__device__ __forceinline__ bool pa_visible(int p, int key, int mask, int size, int keep_first) {
     if (key > p) return false;
-    if (mask == 1) return p - key < size;
+    if (mask == 1) return p - key < size || key < keep_first;
     if (mask == 2) return p / size == key / size;
     return true;
 }
@@ -36,7 +37,7 @@ template <typename T, int VL /* ceil(dv / 32) */>
 __global__ void __launch_bounds__(kPaWarps * 32)
 paged_attention_kernel(const T *__restrict__ q, long long q_token, long long q_head, const T *__restrict__ slab, int num_pages, int page_size,
                        int row_width, int dk, int dv, int heads, int kv_heads, const int32_t *__restrict__ block_table, int max_pages,
-                       const int32_t *__restrict__ tiles, const int32_t *__restrict__ tok_pos, int mask, int mask_size, float scale, float softcap,
+                       const int32_t *__restrict__ tiles, const int32_t *__restrict__ tok_pos, int mask, int mask_size, int keep_first, float scale, float softcap,
                        int sink, const T *__restrict__ gate, long long g_token, T *__restrict__ out, long long o_token, long long o_head,
                        const float *__restrict__ head_bias, int weights) {
     extern __shared__ float smem[];
@@ -80,10 +81,12 @@ paged_attention_kernel(const T *__restrict__ q, long long q_token, long long q_h
     if (mask == 1) lo = max(0, pos0 - mask_size + 1);
     if (mask == 2) lo = pos0 / mask_size * mask_size;
     lo = lo / kPaKeys * kPaKeys;
+    // the kept first positions that the window does not reach are whole tiles ahead of `lo`
+    const int kept = mask == 1 ? min(lo, (keep_first + kPaKeys - 1) / kPaKeys * kPaKeys) : 0;
     const int32_t *table = block_table + (size_t)seq * max_pages;
     const size_t k_off = (size_t)g * dk, v_off = (size_t)kv_heads * dk + (size_t)g * dv;
 
-    for (int k0 = lo; k0 <= hi; k0 += kPaKeys) {
+    for (int k0 = kept > 0 ? 0 : lo; k0 <= hi; k0 = k0 + kPaKeys == kept ? lo : k0 + kPaKeys) {
         __syncthreads();
         int page = table[k0 / page_size];
         bool page_ok = page >= 0 && page < num_pages;
@@ -109,8 +112,8 @@ paged_attention_kernel(const T *__restrict__ q, long long q_token, long long q_h
             s1 = fmaf(qb[d], kv, s1);
         }
         if (softcap > 0.f) s0 = softcap * tanhf(s0 / softcap), s1 = softcap * tanhf(s1 / softcap);
-        bool vis0 = live0 && key <= hi && pa_visible(p0, key, mask, mask_size);
-        bool vis1 = live1 && key <= hi && pa_visible(p1, key, mask, mask_size);
+        bool vis0 = live0 && key <= hi && pa_visible(p0, key, mask, mask_size, keep_first);
+        bool vis1 = live1 && key <= hi && pa_visible(p1, key, mask, mask_size, keep_first);
         float e0, e1;
         if (weights == 1) {
             e0 = vis0 ? 1.0f / (1.0f + expf(-(s0 + hb0))) : 0.f;
@@ -315,7 +318,7 @@ qk_whole_prepare_kernel(T *q, long long q_token, int heads, const T *__restrict_
 template <typename T, int VL>
 static int pa_launch(const void *q, long long q_token, long long q_head, const void *slab, int num_pages, int page_size, int dk, int dv, int heads,
                      int kv_heads, const int32_t *block_table, int max_pages, const int32_t *tiles, int num_tiles, const int32_t *tok_pos, int mask,
-                     int mask_size, float scale, float softcap, int sink, const void *gate, long long g_token, void *out, long long o_token,
+                     int mask_size, int keep_first, float scale, float softcap, int sink, const void *gate, long long g_token, void *out, long long o_token,
                      long long o_head, const float *head_bias, int weights, cudaStream_t st) {
     size_t smem = ((size_t)kPaRows * dk + (size_t)kPaKeys * (dk + 1) + (size_t)kPaKeys * dv) * sizeof(float);
     auto kernel = paged_attention_kernel<T, VL>;
@@ -327,7 +330,7 @@ static int pa_launch(const void *q, long long q_token, long long q_head, const v
     int group = heads / kv_heads;
     dim3 grid(num_tiles, kv_heads * ceil_div(group, pa_heads_per_cta(group)));
     kernel<<<grid, kPaWarps * 32, smem, st>>>((const T *)q, q_token, q_head, (const T *)slab, num_pages, page_size, kv_heads * (dk + dv), dk, dv, heads,
-                                              kv_heads, block_table, max_pages, tiles, tok_pos, mask, mask_size, scale, softcap, sink, (const T *)gate,
+                                              kv_heads, block_table, max_pages, tiles, tok_pos, mask, mask_size, keep_first, scale, softcap, sink, (const T *)gate,
                                               g_token, (T *)out, o_token, o_head, head_bias, weights);
     return TL_OK;
 }
@@ -345,7 +348,7 @@ int tlb_paged_attention_tile_tokens(int heads, int kv_heads) {
 
 int tlb_paged_attention(const void *q, long long q_token, long long q_head, const void *slab, int num_pages, int page_size, int dk, int dv, int heads,
                         int kv_heads, const int32_t *block_table, int max_pages, const int32_t *tiles, int num_tiles, const int32_t *tok_pos, int mask,
-                        int mask_size, float scale, float softcap, int sink, const void *gate, long long g_token, void *out, long long o_token,
+                        int mask_size, int keep_first, float scale, float softcap, int sink, const void *gate, long long g_token, void *out, long long o_token,
                         long long o_head, const float *head_bias, int weights, int dtype, void *stream) {
     if (num_tiles <= 0) return TL_OK;
     if (weights < 0 || weights > 1 || (weights == 1 && (sink || softcap > 0.f))) return tl::fail(TL_EINVAL, "paged_attention: bad weights mode");
@@ -353,14 +356,15 @@ int tlb_paged_attention(const void *q, long long q_token, long long q_head, cons
         max_pages <= 0 || num_pages <= 0)
         return tl::fail(TL_EINVAL, "paged_attention: bad argument");
     if (page_size <= 0 || page_size % kPaKeys != 0) return tl::fail(TL_EINVAL, "paged_attention: page_size must be a multiple of %d", kPaKeys);
-    if (mask < 0 || mask > 2 || (mask != 0 && mask_size <= 0)) return tl::fail(TL_EINVAL, "paged_attention: bad mask");
+    if (mask < 0 || mask > 2 || (mask != 0 && mask_size <= 0) || keep_first < 0 || keep_first > (1 << 30) || (keep_first > 0 && mask != 1))
+        return tl::fail(TL_EINVAL, "paged_attention: bad mask");
     if (dv > 512) return tl::fail(TL_EINVAL, "paged_attention: value size %d > 512", dv);
     cudaStream_t st = as_stream(stream);
     int vl = ceil_div(dv, 32);
     int rc = TL_OK;
 #define TLB_PA(V)                                                                                                                                   \
     rc = pa_launch<T, V>(q, q_token, q_head, slab, num_pages, page_size, dk, dv, heads, kv_heads, block_table, max_pages, tiles, num_tiles, tok_pos, \
-                         mask, mask_size, scale, softcap, sink, gate, g_token, out, o_token, o_head, head_bias, weights, st)
+                         mask, mask_size, keep_first, scale, softcap, sink, gate, g_token, out, o_token, o_head, head_bias, weights, st)
     TLB_DISPATCH(dtype, "paged_attention", if (vl <= 1) TLB_PA(1); else if (vl <= 2) TLB_PA(2); else if (vl <= 4) TLB_PA(4); else if (vl <= 8) TLB_PA(8);
                  else TLB_PA(16));
 #undef TLB_PA

@@ -60,7 +60,7 @@ __global__ void __launch_bounds__(kGWarps * 32)
 paged_attention_mma_kernel(const bf16 *__restrict__ q, long long q_token, long long q_head, const bf16 *__restrict__ slab, int num_pages, int page_size,
                            int row_width, int dk, int dv, int heads, int kv_heads, int hp /* query heads per CTA */,
                            const int32_t *__restrict__ block_table, int max_pages, const int32_t *__restrict__ tiles, const int32_t *__restrict__ tok_pos,
-                           int mask, int mask_size, float scale, float softcap, int sink, const bf16 *__restrict__ gate, long long g_token,
+                           int mask, int mask_size, int keep_first, float scale, float softcap, int sink, const bf16 *__restrict__ gate, long long g_token,
                            bf16 *__restrict__ out, long long o_token, long long o_head, int k_stride, int v_stride /* shared-memory row strides */,
                            float *__restrict__ partial /* split results, or NULL */, const float *__restrict__ head_bias /* [heads] or NULL */,
                            int weights /* 0 softmax, 1 sigmoid(score + head_bias) without normalisation */) {
@@ -100,7 +100,10 @@ paged_attention_mma_kernel(const bf16 *__restrict__ q, long long q_token, long l
     if (mask == 2) lo = pos0 / mask_size * mask_size;
     lo = lo / kGKeys * kGKeys;
     const int32_t *table = block_table + (size_t)seq * max_pages;
-    const int n_tiles = (hi - lo) / kGKeys + 1;
+    // the kept first positions that the window does not reach are whole key tiles ahead of those from `lo` on
+    const int kept_tiles = mask == 1 ? min(lo, (keep_first + kGKeys - 1) / kGKeys * kGKeys) / kGKeys : 0;
+    const int n_tiles = kept_tiles + (hi - lo) / kGKeys + 1;
+    auto tile_key = [&](int tile) { return tile < kept_tiles ? tile * kGKeys : lo + (tile - kept_tiles) * kGKeys; };  // a tile's first key
     const size_t k_off = (size_t)g * dk, v_off = (size_t)kv_heads * dk + (size_t)g * dv;
 
     // which 16-byte piece of which row this thread copies first (the same for every tile); the next ones are 256 pieces on
@@ -108,7 +111,7 @@ paged_attention_mma_kernel(const bf16 *__restrict__ q, long long q_token, long l
     const int step_rows = (int)blockDim.x / per_row, step_pieces = (int)blockDim.x % per_row;
     auto stage = [&](int tile, int buf) {
         bf16 *sk = skv + buf * buf_elems, *sv = sk + kGKeys * k_stride;
-        int k0 = lo + tile * kGKeys;
+        int k0 = tile_key(tile);
         int page = table[k0 / page_size];
         bool ok = page >= 0 && page < num_pages;
         int valid = ok ? min(kGKeys, hi - k0 + 1) : 0;
@@ -130,7 +133,7 @@ paged_attention_mma_kernel(const bf16 *__restrict__ q, long long q_token, long l
     const bool sunk = sink && blockIdx.z == 0;  // with the key range split over gridDim.z CTAs the sink's term is counted once
     float m_row = sunk ? 0.f : -INFINITY, l_row = sunk ? 1.f : 0.f;
     float hb = 0.f;  // the row's head's learned number: the sink's score, or the offset inside the sigmoid
-    int see_lo = 1, see_hi = 0;  // the keys this row may see (none for a padding row)
+    int see_lo = 1, see_hi = 0, see_first = 0;  // the keys this row may see: [see_lo, see_hi] and those below see_first (none for a padding row)
     {
         int r = warp * 4 + (lane >> 3), tq = r / hp, hh = r % hp;
         if (tq < count && hh < nheads) {
@@ -138,6 +141,7 @@ paged_attention_mma_kernel(const bf16 *__restrict__ q, long long q_token, long l
             if (sunk) m_row = hb;
             if (weights == 1) m_row = 0.f, l_row = blockIdx.z == 0 ? 1.f : 0.f;
             see_hi = pos0 + tq;
+            see_first = mask == 1 ? keep_first : 0;
             see_lo = mask == 1 ? max(0, see_hi - mask_size + 1) : mask == 2 ? see_hi / mask_size * mask_size : 0;
         }
     }
@@ -190,13 +194,13 @@ paged_attention_mma_kernel(const bf16 *__restrict__ q, long long q_token, long l
         // 2. softmax over this tile's keys: a warp owns 4 rows, 8 lanes per row, 4 keys per lane (keys lq + 8 j)
         {
             const int i = lane >> 3, lq = lane & 7, r = warp * 4 + i;
-            const int key0 = lo + tile * kGKeys + lq;
+            const int key0 = tile_key(tile) + lq;
             float sv4[kGKeys / 8];
             float mx = -INFINITY;
 #pragma unroll
             for (int j = 0; j < kGKeys / 8; ++j) {
                 int key = key0 + 8 * j;
-                bool vis = key >= see_lo && key <= see_hi;
+                bool vis = (key >= see_lo || key < see_first) && key <= see_hi;
                 float s = ss[r * kGSS + lq + 8 * j];
                 if (softcap > 0.f) s = softcap * g_tanh(s * inv_cap);
                 sv4[j] = vis ? s : -INFINITY;
@@ -362,7 +366,7 @@ size_t tlb_paged_attention_mma_workspace(int num_tiles, int heads, int kv_heads,
 
 int tlb_paged_attention_mma(const void *q, long long q_token, long long q_head, const void *slab, int num_pages, int page_size, int dk, int dv, int heads,
                             int kv_heads, const int32_t *block_table, int max_pages, const int32_t *tiles, int num_tiles, const int32_t *tok_pos,
-                            int mask, int mask_size, float scale, float softcap, int sink, const void *gate, long long g_token, void *out,
+                            int mask, int mask_size, int keep_first, float scale, float softcap, int sink, const void *gate, long long g_token, void *out,
                             long long o_token, long long o_head, int splits, void *workspace, size_t workspace_bytes, const float *head_bias,
                             int weights, void *stream) {
     if (num_tiles <= 0) return TL_OK;
@@ -371,7 +375,8 @@ int tlb_paged_attention_mma(const void *q, long long q_token, long long q_head, 
         return tl::fail(TL_EINVAL, "paged_attention_mma: bad argument");
     if (!tlb_paged_attention_mma_supported(dk, dv, kv_heads, page_size))
         return tl::fail(TL_EINVAL, "paged_attention_mma: dk, dv multiples of 8 up to 256 and page_size %% 32 == 0 are required");
-    if (mask < 0 || mask > 2 || (mask != 0 && mask_size <= 0)) return tl::fail(TL_EINVAL, "paged_attention_mma: bad mask");
+    if (mask < 0 || mask > 2 || (mask != 0 && mask_size <= 0) || keep_first < 0 || keep_first > (1 << 30) || (keep_first > 0 && mask != 1))
+        return tl::fail(TL_EINVAL, "paged_attention_mma: bad mask");
     if (!tl::aligned16(slab)) return tl::fail(TL_EINVAL, "paged_attention_mma: the cache must be 16-byte aligned");
     int group = heads / kv_heads;
     int hp = group >= kGRows ? kGRows : group;
@@ -394,7 +399,7 @@ int tlb_paged_attention_mma(const void *q, long long q_token, long long q_head, 
             if (e != cudaSuccess) return tl::fail(TL_ECUDA, "paged_attention_mma: %s", cudaGetErrorString(e));                                   \
         }                                                                                                                                        \
         kernel<<<grid, kGWarps * 32, smem, st>>>((const bf16 *)q, q_token, q_head, (const bf16 *)slab, num_pages, page_size, kv_heads * (dk + dv), dk, dv, \
-                                                 heads, kv_heads, hp, block_table, max_pages, tiles, tok_pos, mask, mask_size, scale, softcap, sink,    \
+                                                 heads, kv_heads, hp, block_table, max_pages, tiles, tok_pos, mask, mask_size, keep_first, scale, softcap, sink, \
                                                  (const bf16 *)gate, g_token, (bf16 *)out, o_token, o_head, k_stride, v_stride, part, head_bias, weights); \
     } while (0)
     if (pairs == 1) TLB_PAM(1);

@@ -4,6 +4,7 @@
 #include <stdio.h>
 
 #include <atomic>
+#include <initializer_list>
 
 #include "blocks_common.cuh"
 
@@ -121,24 +122,106 @@ __global__ void norm_residual_kernel(const TY *__restrict__ y, const T *__restri
 }
 
 
-// residual += a (+ b) in fp32, then (w != NULL) h = residual / rms(residual) * w rounded to T: the end of a sublayer (or of
-// a layer whose sublayers both read one norm of the stream), fused with the norm that reads the stream next.  a_row: `a`
-// is ONE row [dim] added to every row (a learned offset).
-template <typename T>
-__global__ void add_norm_kernel(float *__restrict__ residual, const float *__restrict__ a, int a_row, const float *__restrict__ b,
-                                const T *__restrict__ w, float eps, T *__restrict__ h, int dim) {
-    __shared__ float scratch[33];
-    size_t base = (size_t)blockIdx.x * dim, abase = a_row ? 0 : base;
+// A new row of the fp32 residual stream and the norms that read it next, a CTA per row: `make4(q)` / `make1(d)` give columns
+// 4 q .. 4 q + 3 / column d of the new row, which goes to `row`; then (h1 != NULL) h1 = row / rms(row) * w1 and (h2 != NULL)
+// h2 = row / rms(row) * w2, rounded to T.  VEC: 16-byte accesses (dim % 4 == 0, aligned bases), the row kept in registers
+// between the two sweeps when it has at most 4 * KEEP * blockDim columns.
+template <typename T, bool VEC, typename Make4, typename Make1>
+__device__ __forceinline__ void stream_row(Make4 make4, Make1 make1, float *row, const T *__restrict__ w1, T *h1, const T *__restrict__ w2, T *h2,
+                                           float eps, int dim, float *scratch) {
     float ss = 0.f;
-    for (int d = threadIdx.x; d < dim; d += blockDim.x) {
-        float x = residual[base + d] + (b ? a[abase + d] + b[base + d] : a[abase + d]);
-        residual[base + d] = x;
-        ss += x * x;
+    if constexpr (VEC) {
+        constexpr int KEEP = 4;
+        float4 kept[KEEP];
+        const int quads = dim / 4;
+        auto take = [&](int q) {
+            float4 v = make4(q);
+            store4(row + 4 * q, v);
+            ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+            return v;
+        };
+#pragma unroll
+        for (int i = 0; i < KEEP; ++i) {
+            int q = threadIdx.x + i * blockDim.x;
+            if (q < quads) kept[i] = take(q);
+        }
+        for (int q = threadIdx.x + KEEP * blockDim.x; q < quads; q += blockDim.x) take(q);
+        if (h1 == nullptr) return;
+        ss = block_sum(ss, scratch);
+        const float inv = 1.0f / sqrtf(ss / (float)dim + eps);
+        auto give = [&](int q, float4 v) {
+            v.x *= inv, v.y *= inv, v.z *= inv, v.w *= inv;
+            float4 g = load4(w1 + 4 * q);
+            store4(h1 + 4 * q, make_float4(v.x * g.x, v.y * g.y, v.z * g.z, v.w * g.w));
+            if (h2 == nullptr) return;
+            g = load4(w2 + 4 * q);
+            store4(h2 + 4 * q, make_float4(v.x * g.x, v.y * g.y, v.z * g.z, v.w * g.w));
+        };
+#pragma unroll
+        for (int i = 0; i < KEEP; ++i) {
+            int q = threadIdx.x + i * blockDim.x;
+            if (q < quads) give(q, kept[i]);
+        }
+        for (int q = threadIdx.x + KEEP * blockDim.x; q < quads; q += blockDim.x) give(q, load4(row + 4 * q));
+    } else {
+        for (int d = threadIdx.x; d < dim; d += blockDim.x) {
+            float x = make1(d);
+            row[d] = x;
+            ss += x * x;
+        }
+        if (h1 == nullptr) return;
+        ss = block_sum(ss, scratch);
+        const float inv = 1.0f / sqrtf(ss / (float)dim + eps);
+        for (int d = threadIdx.x; d < dim; d += blockDim.x) {
+            float x = row[d] * inv;
+            h1[d] = from_f<T>(x * to_f(w1[d]));
+            if (h2 != nullptr) h2[d] = from_f<T>(x * to_f(w2[d]));
+        }
     }
-    if (w == nullptr || h == nullptr) return;
-    ss = block_sum(ss, scratch);
-    float inv = 1.0f / sqrtf(ss / (float)dim + eps);
-    for (int d = threadIdx.x; d < dim; d += blockDim.x) h[base + d] = from_f<T>(residual[base + d] * inv * to_f(w[d]));
+}
+
+__device__ __forceinline__ float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
+
+// residual += a (+ b) in fp32, then the norms that read the stream next (w: one, w2: a second one with its own weights): the
+// end of a sublayer, or of a layer whose sublayers both read the stream as it was.  a_row: `a` is ONE row [dim] added to
+// every row (a learned offset).
+template <typename T, bool VEC>
+__global__ void add_norm_kernel(float *__restrict__ residual, const float *__restrict__ a, int a_row, const float *__restrict__ b,
+                                const T *__restrict__ w, float eps, T *__restrict__ h, const T *__restrict__ w2, T *__restrict__ h2, int dim) {
+    __shared__ float scratch[33];
+    const size_t base = (size_t)blockIdx.x * dim, abase = a_row ? 0 : base;
+    float *row = residual + base;
+    stream_row<T, VEC>([&](int q) { return add4(load4(row + 4 * q), b ? add4(load4(a + abase + 4 * q), load4(b + base + 4 * q)) : load4(a + abase + 4 * q)); },
+                       [&](int d) { return row[d] + (b ? a[abase + d] + b[base + d] : a[abase + d]); }, row, w, h ? h + base : nullptr, w2,
+                       h2 ? h2 + base : nullptr, eps, dim, scratch);
+}
+
+// The start of the residual stream: x = table[id] * scale (+ pairs[row], row = (id before * mul_prev + id * mul_cur) mod buckets,
+// the table's last row for a sequence's first token), then the norms that read it.  The token before is the flat batch's
+// when it belongs to the same sequence, else the one the sequence ended its last step with (seq_prev[seq]).
+template <typename T, bool VEC>
+__global__ void embed_pairs_kernel(const int32_t *__restrict__ ids, const int32_t *__restrict__ tok_pos, const int32_t *__restrict__ tok_seq,
+                                   const int32_t *__restrict__ seq_prev, const T *__restrict__ table, int vocab, float scale, const T *__restrict__ pairs,
+                                   long long buckets, long long mul_prev, long long mul_cur, float *__restrict__ x32, const T *__restrict__ w1,
+                                   T *__restrict__ h1, const T *__restrict__ w2, T *__restrict__ h2, float eps, int dim) {
+    __shared__ float scratch[33];
+    const int t = blockIdx.x;
+    const int id = ids[t];
+    const T *e = table + (size_t)(id < 0 || id >= vocab ? 0 : id) * dim;
+    const T *g = nullptr;
+    if (pairs != nullptr) {
+        long long bucket = buckets;
+        if (tok_pos[t] > 0) {
+            const int before = t > 0 && tok_seq[t - 1] == tok_seq[t] ? ids[t - 1] : seq_prev[tok_seq[t]];
+            if (before >= 0 && id >= 0) bucket = (before * mul_prev + id * mul_cur) % buckets;
+        }
+        g = pairs + (size_t)bucket * dim;
+    }
+    auto scaled = [&](float4 v) { return make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale); };
+    const size_t base = (size_t)t * dim;
+    stream_row<T, VEC>([&](int q) { float4 v = scaled(load4(e + 4 * q)); return g ? add4(v, load4(g + 4 * q)) : v; },
+                       [&](int d) { float v = to_f(e[d]) * scale; return g ? v + to_f(g[d]) : v; }, x32 + base, w1, h1 ? h1 + base : nullptr, w2,
+                       h2 ? h2 + base : nullptr, eps, dim, scratch);
 }
 
 // y = coef * (a / rms(a) * wa + b / rms(b) * wb), fp32 in and out: two mixers side by side, each normed before they meet.
@@ -269,16 +352,17 @@ __device__ __forceinline__ float gated_pair(float g, float u, int act, float lim
 }
 
 template <typename T>
-__global__ void gated_act_kernel(const T *__restrict__ gu, T *__restrict__ out, long long total, int width, int act, float limit, float slope) {
+__global__ void gated_act_kernel(const T *__restrict__ gu, T *__restrict__ out, long long out_row, long long total, int width, int act, float limit, float slope) {
     long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= total) return;
     long long row = i / width;
     int j = (int)(i - row * width);
-    out[i] = from_f<T>(gated_pair(to_f(gu[row * 2 * width + j]), to_f(gu[row * 2 * width + width + j]), act, limit, slope));
+    out[row * out_row + j] = from_f<T>(gated_pair(to_f(gu[row * 2 * width + j]), to_f(gu[row * 2 * width + width + j]), act, limit, slope));
 }
 
 // Eight adjacent columns per thread, 16-byte accesses (bf16, width % 8 == 0).
-__global__ void gated_act_wide_kernel(const bf16 *__restrict__ gu, bf16 *__restrict__ out, long long total8, int width, int act, float limit, float slope) {
+__global__ void gated_act_wide_kernel(const bf16 *__restrict__ gu, bf16 *__restrict__ out, long long out_row, long long total8, int width, int act, float limit,
+                                      float slope) {
     long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= total8) return;
     const int per_row = width / 8;
@@ -292,7 +376,7 @@ __global__ void gated_act_wide_kernel(const bf16 *__restrict__ gu, bf16 *__restr
         float2 g = __bfloat1622float2(gp[e]), u = __bfloat1622float2(up[e]);
         op[e] = __floats2bfloat162_rn(gated_pair(g.x, u.x, act, limit, slope), gated_pair(g.y, u.y, act, limit, slope));
     }
-    *reinterpret_cast<uint4 *>(out + row * width + j) = o4;
+    *reinterpret_cast<uint4 *>(out + row * out_row + j) = o4;
 }
 
 __global__ void argmax_rows_kernel(const float *__restrict__ logits, int32_t *__restrict__ out, int vocab) {
@@ -332,7 +416,7 @@ using namespace tlb;
 
 extern "C" {
 
-int tlb_abi_version(void) { return 5; }
+int tlb_abi_version(void) { return 6; }
 const char *tlb_last_error(void) { return tl::g_error; }
 long long tlb_launch_count(void) { return tl::g_launches.load(std::memory_order_relaxed); }
 
@@ -363,13 +447,44 @@ int tlb_norm_residual(const void *y, int y_is_f32, const void *w, float weight_o
     return TL_OK;
 }
 
-int tlb_add_norm(float *residual, const float *a, int a_row, const float *b, const void *w, float eps, void *h, int rows, int dim, int dtype,
-                 void *stream) {
+static bool rows_aligned(int dim, std::initializer_list<const void *> bases) {
+    if (dim % 4) return false;
+    for (const void *p : bases)
+        if (p && !tl::aligned16(p)) return false;
+    return true;
+}
+
+int tlb_add_norm(float *residual, const float *a, int a_row, const float *b, const void *w, float eps, void *h, const void *w2, void *h2, int rows,
+                 int dim, int dtype, void *stream) {
     if (rows <= 0) return TL_OK;
-    if (!residual || !a || dim <= 0 || ((w == nullptr) != (h == nullptr))) return tl::fail(TL_EINVAL, "add_norm: bad argument");
+    if (!residual || !a || dim <= 0 || ((w == nullptr) != (h == nullptr)) || ((w2 == nullptr) != (h2 == nullptr)) || (w2 && !w))
+        return tl::fail(TL_EINVAL, "add_norm: bad argument");
     int threads = dim >= 2048 ? 256 : 128;
-    TLB_DISPATCH(dtype, "add_norm", add_norm_kernel<T><<<rows, threads, 0, as_stream(stream)>>>(residual, a, a_row, b, (const T *)w, eps, (T *)h, dim));
+    const bool vec = rows_aligned(dim, {residual, a, b, w, h, w2, h2});
+#define TLB_ADD_NORM(V) add_norm_kernel<T, V><<<rows, threads, 0, as_stream(stream)>>>(residual, a, a_row, b, (const T *)w, eps, (T *)h, (const T *)w2, (T *)h2, dim)
+    TLB_DISPATCH(dtype, "add_norm", if (vec) TLB_ADD_NORM(true); else TLB_ADD_NORM(false));
+#undef TLB_ADD_NORM
     TL_LAUNCH_CHECK("add_norm");
+    return TL_OK;
+}
+
+int tlb_embed_pairs(const int32_t *ids, const int32_t *tok_pos, const int32_t *tok_seq, const int32_t *seq_prev, const void *table, int vocab, float scale,
+                    const void *pairs, long long buckets, long long mul_prev, long long mul_cur, float *x32, const void *w1, void *h1, const void *w2,
+                    void *h2, float eps, int tokens, int dim, int dtype, void *stream) {
+    if (tokens <= 0) return TL_OK;
+    if (!ids || !table || !x32 || vocab <= 0 || dim <= 0 || ((w1 == nullptr) != (h1 == nullptr)) || ((w2 == nullptr) != (h2 == nullptr)) || (w2 && !w1))
+        return tl::fail(TL_EINVAL, "embed_pairs: bad argument");
+    // the multipliers are residues: with ids below 2^31 the sum of both products stays below 2^63
+    if (pairs && (!tok_pos || !tok_seq || !seq_prev || buckets <= 0 || buckets >= (1LL << 31) || mul_prev < 0 || mul_prev >= buckets || mul_cur < 0 || mul_cur >= buckets))
+        return tl::fail(TL_EINVAL, "embed_pairs: bad pair table");
+    int threads = dim >= 2048 ? 256 : 128;
+    const bool vec = rows_aligned(dim, {table, pairs, x32, w1, h1, w2, h2});
+#define TLB_EMBED(V)                                                                                                                                \
+    embed_pairs_kernel<T, V><<<tokens, threads, 0, as_stream(stream)>>>(ids, tok_pos, tok_seq, seq_prev, (const T *)table, vocab, scale, (const T *)pairs, \
+                                                                        buckets, mul_prev, mul_cur, x32, (const T *)w1, (T *)h1, (const T *)w2, (T *)h2, eps, dim)
+    TLB_DISPATCH(dtype, "embed_pairs", if (vec) TLB_EMBED(true); else TLB_EMBED(false));
+#undef TLB_EMBED
+    TL_LAUNCH_CHECK("embed_pairs");
     return TL_OK;
 }
 
@@ -421,16 +536,16 @@ int tlb_latent_prepare(const void *down, long long down_stride, const void *norm
     return TL_OK;
 }
 
-int tlb_gated_act(const void *gu, void *out, int rows, int width, int act, float limit, float slope, int dtype, void *stream) {
+int tlb_gated_act(const void *gu, void *out, long long out_row, int rows, int width, int act, float limit, float slope, int dtype, void *stream) {
     if (rows <= 0 || width <= 0) return TL_OK;
-    if (!gu || !out || (act != 0 && act != 1 && act != 3) || (act == 3 && !(limit > 0.f))) return tl::fail(TL_EINVAL, "gated_act: bad argument");
+    if (!gu || !out || (act != 0 && act != 1 && act != 3) || (act == 3 && !(limit > 0.f)) || out_row < width) return tl::fail(TL_EINVAL, "gated_act: bad argument");
     long long total = (long long)rows * width;
-    if (dtype == TL_BF16 && width % 8 == 0 && (uintptr_t)gu % 16 == 0 && (uintptr_t)out % 16 == 0) {
+    if (dtype == TL_BF16 && width % 8 == 0 && out_row % 8 == 0 && (uintptr_t)gu % 16 == 0 && (uintptr_t)out % 16 == 0) {
         long long total8 = total / 8;
-        gated_act_wide_kernel<<<(unsigned)((total8 + 255) / 256), 256, 0, as_stream(stream)>>>((const bf16 *)gu, (bf16 *)out, total8, width, act, limit, slope);
+        gated_act_wide_kernel<<<(unsigned)((total8 + 255) / 256), 256, 0, as_stream(stream)>>>((const bf16 *)gu, (bf16 *)out, out_row, total8, width, act, limit, slope);
     } else
         TLB_DISPATCH(dtype, "gated_act",
-                     gated_act_kernel<T><<<(unsigned)((total + 255) / 256), 256, 0, as_stream(stream)>>>((const T *)gu, (T *)out, total, width, act, limit, slope));
+                     gated_act_kernel<T><<<(unsigned)((total + 255) / 256), 256, 0, as_stream(stream)>>>((const T *)gu, (T *)out, out_row, total, width, act, limit, slope));
     TL_LAUNCH_CHECK("gated_act");
     return TL_OK;
 }

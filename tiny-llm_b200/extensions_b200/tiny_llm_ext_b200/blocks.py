@@ -25,9 +25,10 @@ _SIGNATURES = {
     "tlb_last_error": (ctypes.c_char_p, []),
     "tlb_launch_count": (_LL, []),
     "tlb_embed_rows": (_I, [_VP, _VP, _VP, _VP, _I, _I, _I, _I, _VP]),
+    "tlb_embed_pairs": (_I, [_VP, _VP, _VP, _VP, _VP, _I, _F, _VP, _LL, _LL, _LL, _VP, _VP, _VP, _VP, _VP, _F, _I, _I, _I, _VP]),
     "tlb_norm_residual": (_I, [_VP, _I, _VP, _F, _VP, _F, _VP, _VP, _I, _I, _I, _VP]),
     "tlb_rope_rows": (_I, [_VP, _LL, _LL, _I, _I, _I, _I, _D, _D, _VP, _I, _I, _VP]),
-    "tlb_rope_table": (_I, [_VP, _I, _I, _D, _D, _VP, _VP, _VP]),
+    "tlb_rope_table": (_I, [_VP, _I, _I, _D, _D, _D, _D, _D, _D, _VP, _VP, _VP]),
     "tlb_latent_append": (_I, [_VP, _VP, _F, _I, _I, _I, _I, _D, _VP, _VP, _VP, _I, _I, _I, _VP, _I, _I, _VP]),
     "tlb_latent_prepare": (_I, [_VP, _LL, _VP, _F, _I, _I, _I, _I, _D, _VP, _VP, _VP, _I, _I, _I, _VP, _VP, _LL, _I, _I, _I, _I, _I, _VP]),
     "tlb_latent_attention": (_I, [_VP, _LL, _LL, _VP, _LL, _LL, _VP, _I, _I, _I, _I, _VP, _I, _VP, _I, _VP, _I, _I, _F, _VP, _LL, _LL, _VP, _I, _VP]),
@@ -36,20 +37,20 @@ _SIGNATURES = {
     "tlb_latent_attention_mma": (_I, [_VP, _LL, _LL, _VP, _LL, _LL, _VP, _I, _I, _I, _I, _VP, _I, _VP, _I, _VP, _I, _I, _F, _VP, _LL, _LL, _I, _VP,
                                       ctypes.c_size_t, _VP, _VP]),
     "tlb_latent_attention_mma_workspace": (ctypes.c_size_t, [_I, _I, _I, _I]),
-    "tlb_gated_act": (_I, [_VP, _VP, _I, _I, _I, _F, _F, _I, _VP]),
+    "tlb_gated_act": (_I, [_VP, _VP, _LL, _I, _I, _I, _F, _F, _I, _VP]),
     "tlb_streams_step": (_I, [_VP, _VP, _VP, _VP, _VP, _VP, _F, _VP, _I, _I, _I, _I, _VP]),
     "tlb_shift_mix": (_I, [_VP, _LL, _VP, _I, _I, _VP, _I, _I, _VP, _LL, _I, _VP, _LL, _I, _VP]),
     "tlb_moe_route": (_I, [_VP, _VP, _VP, _I, _I, _I, _I, _I, _VP, _F, _VP, _VP, _I, _VP]),
     "tlb_moe_up": (_I, [_VP, _VP, _VP, _VP, _VP, _I, _I, _I, _I, _I, _I, _I, _I, _VP, _I, _VP]),
     "tlb_moe_scale_rows": (_I, [_VP, _VP, _VP, _I, _I, _I, _I, _VP]),
-    "tlb_add_norm": (_I, [_VP, _VP, _I, _VP, _VP, _F, _VP, _I, _I, _I, _VP]),
+    "tlb_add_norm": (_I, [_VP, _VP, _I, _VP, _VP, _F, _VP, _VP, _VP, _I, _I, _I, _VP]),
     "tlb_norm_mix2": (_I, [_VP, _VP, _VP, _VP, _F, _F, _VP, _I, _I, _I, _VP]),
     "tlb_paged_attention_tile_tokens": (_I, [_I, _I]),
-    "tlb_paged_attention": (_I, [_VP, _LL, _LL, _VP, _I, _I, _I, _I, _I, _I, _VP, _I, _VP, _I, _VP, _I, _I, _F, _F, _I, _VP, _LL, _VP, _LL, _LL, _VP, _I, _I,
+    "tlb_paged_attention": (_I, [_VP, _LL, _LL, _VP, _I, _I, _I, _I, _I, _I, _VP, _I, _VP, _I, _VP, _I, _I, _I, _F, _F, _I, _VP, _LL, _VP, _LL, _LL, _VP, _I, _I,
                                  _VP]),
     "tlb_paged_attention_mma_tile_tokens": (_I, [_I, _I]),
     "tlb_paged_attention_mma_supported": (_I, [_I, _I, _I, _I]),
-    "tlb_paged_attention_mma": (_I, [_VP, _LL, _LL, _VP, _I, _I, _I, _I, _I, _I, _VP, _I, _VP, _I, _VP, _I, _I, _F, _F, _I, _VP, _LL, _VP, _LL, _LL, _I, _VP,
+    "tlb_paged_attention_mma": (_I, [_VP, _LL, _LL, _VP, _I, _I, _I, _I, _I, _I, _VP, _I, _VP, _I, _VP, _I, _I, _I, _F, _F, _I, _VP, _LL, _VP, _LL, _LL, _I, _VP,
                                      ctypes.c_size_t, _VP, _I, _VP]),
     "tlb_paged_attention_mma_workspace": (ctypes.c_size_t, [_I, _I, _I, _I, _I]),
     "tlb_kv_prepare": (_I, [_VP, _LL, _LL, _I, _VP, _VP, _LL, _LL, _VP, _LL, _LL, _I, _I, _I, _VP, _F, _VP, _VP, _VP, _I, _I, _I, _VP, _I, _I, _VP]),
@@ -74,7 +75,7 @@ _SIGNATURES = {
 }
 EXPORTED_SYMBOLS = tuple(_SIGNATURES)
 
-ABI_VERSION = 5
+ABI_VERSION = 6
 ATTENTION_TILE_TOKENS = 4
 MOE_TILE_ROWS = 32
 ACT_SILU, ACT_GELU_TANH, ACT_RELU_SQUARED, ACT_CLAMPED_SWISH, ACT_TANH = 0, 1, 2, 3, 4
@@ -178,6 +179,35 @@ def embed_rows(ids: torch.Tensor, table: torch.Tensor):
     return x32, h
 
 
+def embed_pairs(ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0, *, pairs=None, mul_prev: int = 0, mul_cur: int = 0, tok_pos=None, tok_seq=None,
+                seq_prev=None, weight=None, weight2=None, eps: float = 0.0):
+    """The start of the residual stream: ``table[id] * scale``, plus (``pairs [buckets + 1, D]``) the row
+    ``(previous id * mul_prev + id * mul_cur) mod buckets`` - the last one for a sequence's first token - and the RMS norms
+    that read it first (``weight``, ``weight2``).  ``seq_prev [S]`` int32: the token every sequence ended its last step with.
+    -> (x32 [T, D] fp32, norm or None, second norm or None)."""
+    _gpu("embed_pairs", ids, table, pairs, tok_pos, tok_seq, seq_prev, weight, weight2)
+    _contig("embed_pairs", ids, table, pairs, tok_pos, tok_seq, seq_prev, weight, weight2)
+    if ids.dtype != torch.int32 or ids.dim() != 1 or table.dim() != 2:
+        raise RuntimeError("embed_pairs: ids must be int32 [T] and table [vocab, dim]")
+    T, (V, D) = ids.numel(), table.shape
+    buckets = 0
+    if pairs is not None:
+        buckets = pairs.shape[0] - 1
+        if pairs.dim() != 2 or pairs.shape[1] != D or pairs.dtype != table.dtype or buckets <= 0:
+            raise RuntimeError("embed_pairs: pairs must be [buckets + 1, dim] of the table's dtype")
+        if any(t is None or t.dtype != torch.int32 for t in (tok_pos, tok_seq, seq_prev)) or tok_pos.numel() != T or tok_seq.numel() != T:
+            raise RuntimeError("embed_pairs: int32 positions and sequences per token, and every sequence's previous token")
+        mul_prev, mul_cur = int(mul_prev) % buckets, int(mul_cur) % buckets  # the row is a residue anyway: the products fit in 64 bits
+    if any(w is not None and (w.shape != (D,) or w.dtype != table.dtype) for w in (weight, weight2)) or (weight2 is not None and weight is None):
+        raise RuntimeError("embed_pairs: norm weights must be [dim] of the table's dtype")
+    x32 = torch.empty((T, D), dtype=torch.float32, device=table.device)
+    h, h2 = (None if w is None else torch.empty((T, D), dtype=table.dtype, device=table.device) for w in (weight, weight2))
+    _check(library().tlb_embed_pairs(_ptr(ids), _ptr(tok_pos), _ptr(tok_seq), _ptr(seq_prev), _ptr(table), V, float(scale), _ptr(pairs), buckets, int(mul_prev),
+                                     int(mul_cur), _ptr(x32), _ptr(weight), _ptr(h), _ptr(weight2), _ptr(h2), float(eps), T, D, _code(table.dtype),
+                                     _stream(table)))
+    return x32, h, h2
+
+
 def norm_residual(y, weight, eps: float, *, weight_offset: float = 0.0, scale=None, residual=None, want_h: bool = True):
     """RMS norm of ``y [rows, dim]`` (fp32 or the weight's dtype) times ``weight + weight_offset`` (times ``scale``);
     with ``residual`` (fp32, updated in place) the result is added to it.  Returns the (new residual, or the norm)
@@ -213,15 +243,18 @@ def rope_rows(x: torch.Tensor, tok_pos: torch.Tensor, *, heads: int, head_stride
     return x
 
 
-def rope_table(tok_pos: torch.Tensor, *, dims: int, base: float, factor: float = 1.0):
-    """-> (cos, sin) fp32 ``[rows, dims // 2]`` of ``tok_pos * base^(-2i/dims) / factor``, for kernels that rotate in fp32."""
+def rope_table(tok_pos: torch.Tensor, *, dims: int, base: float, factor: float = 1.0, ramp=None):
+    """-> (cos, sin) fp32 ``[rows, dims // 2]`` of ``tok_pos * base^(-2i/dims) / factor``, for kernels that rotate in fp32.
+    ``ramp`` = (factor, lo, hi, gain): frequency i divided by that factor in the measure ``clamp((i - lo) / max(hi - lo, 0.001),
+    0, 1)``, both tables times ``gain`` (``positional_encoding.yarn_ramp``)."""
     _gpu("rope_table", tok_pos)
     if tok_pos.dtype != torch.int32 or tok_pos.dim() != 1 or not tok_pos.is_contiguous() or dims <= 0 or dims % 2:
         raise RuntimeError("rope_table: tok_pos must be contiguous int32 [rows] and dims even")
     rows = tok_pos.numel()
     cs = torch.empty((rows, dims // 2), dtype=torch.float32, device=tok_pos.device)
     sn = torch.empty_like(cs)
-    _check(library().tlb_rope_table(_ptr(tok_pos), rows, int(dims), float(base), float(factor), _ptr(cs), _ptr(sn), _stream(tok_pos)))
+    ramp_factor, lo, hi, gain = (1.0, 0.0, 0.0, 1.0) if ramp is None else (float(v) for v in ramp)
+    _check(library().tlb_rope_table(_ptr(tok_pos), rows, int(dims), float(base), float(factor), ramp_factor, lo, hi, gain, _ptr(cs), _ptr(sn), _stream(tok_pos)))
     return cs, sn
 
 
@@ -340,14 +373,17 @@ def _mma_ok(rank: int, rot: int, page_size: int) -> bool:
     return os.environ.get("TL_LATENT_MMA", "1") != "0" and bool(library().tlb_latent_attention_mma_supported(rank, rot, page_size))
 
 
-def gated_act(gate_up: torch.Tensor, act: int, limit: float = 0.0, slope: float = 1.0) -> torch.Tensor:
+def gated_act(gate_up: torch.Tensor, act: int, limit: float = 0.0, slope: float = 1.0, out=None) -> torch.Tensor:
     """``act(gate) * up`` of ``[rows, 2 * width]`` (gate columns first).  ``ACT_CLAMPED_SWISH``: ``g = min(gate, limit)``,
-    ``u = clamp(up, -limit, limit)``, ``g sigmoid(slope g) (u + 1)``."""
-    _gpu("gated_act", gate_up)
+    ``u = clamp(up, -limit, limit)``, ``g sigmoid(slope g) (u + 1)``.  ``out``: columns of a wider matrix to write to."""
+    _gpu("gated_act", gate_up, out)
     _contig("gated_act", gate_up)
     rows, two = gate_up.shape
-    out = torch.empty((rows, two // 2), dtype=gate_up.dtype, device=gate_up.device)
-    _check(library().tlb_gated_act(_ptr(gate_up), _ptr(out), rows, two // 2, act, float(limit), float(slope), _code(gate_up.dtype), _stream(gate_up)))
+    if out is None:
+        out = torch.empty((rows, two // 2), dtype=gate_up.dtype, device=gate_up.device)
+    elif out.shape != (rows, two // 2) or out.dtype != gate_up.dtype or out.stride(1) != 1:
+        raise RuntimeError("gated_act: out must be [rows, width] of the input's dtype with unit inner stride")
+    _check(library().tlb_gated_act(_ptr(gate_up), _ptr(out), out.stride(0), rows, two // 2, act, float(limit), float(slope), _code(gate_up.dtype), _stream(gate_up)))
     return out
 
 
@@ -408,19 +444,23 @@ def moe_experts(h, idx, gate, w_gate, w_up, w_down, act: int, shared=None, scale
     return y
 
 
-def add_norm(residual: torch.Tensor, a: torch.Tensor, b: torch.Tensor | None, weight: torch.Tensor | None, eps: float):
+def add_norm(residual: torch.Tensor, a: torch.Tensor, b: torch.Tensor | None, weight: torch.Tensor | None, eps: float, weight2: torch.Tensor | None = None):
     """``residual += a (+ b)`` (all fp32 ``[rows, dim]``, in place; ``a`` may be one row ``[dim]`` for all); with ``weight``
-    also returns the RMS norm of the new residual times ``weight``, rounded to the weight's dtype."""
-    _gpu("add_norm", residual, a, b, weight)
-    _contig("add_norm", residual, a, b, weight)
+    also returns the RMS norm of the new residual times ``weight``, rounded to the weight's dtype; with ``weight2`` too, both
+    that and the norm times ``weight2`` (two sublayers reading the stream side by side)."""
+    _gpu("add_norm", residual, a, b, weight, weight2)
+    _contig("add_norm", residual, a, b, weight, weight2)
     rows, dim = residual.shape
     a_row = a.dim() == 1
     if residual.dtype != torch.float32 or a.dtype != torch.float32 or a.shape != (residual.shape[1:] if a_row else residual.shape) or (b is not None and (b.dtype != torch.float32 or b.shape != residual.shape)):
         raise RuntimeError("add_norm: residual and addends must be float32 of one shape")
-    h = None if weight is None else torch.empty((rows, dim), dtype=weight.dtype, device=residual.device)
+    if any(w is not None and w.shape != (dim,) for w in (weight, weight2)) or (weight2 is not None and (weight is None or weight2.dtype != weight.dtype)):
+        raise RuntimeError("add_norm: norm weights must be [dim] of one dtype")
+    h, h2 = (None if w is None else torch.empty((rows, dim), dtype=w.dtype, device=residual.device) for w in (weight, weight2))
     code = _code(weight.dtype) if weight is not None else 0
-    _check(library().tlb_add_norm(_ptr(residual), _ptr(a), int(a_row), _ptr(b), _ptr(weight), float(eps), _ptr(h), rows, dim, code, _stream(residual)))
-    return h
+    _check(library().tlb_add_norm(_ptr(residual), _ptr(a), int(a_row), _ptr(b), _ptr(weight), float(eps), _ptr(h), _ptr(weight2), _ptr(h2), rows, dim, code,
+                                  _stream(residual)))
+    return h if weight2 is None else (h, h2)
 
 
 def norm_mix2(a: torch.Tensor, wa: torch.Tensor, b: torch.Tensor, wb: torch.Tensor, coef: float, eps: float) -> torch.Tensor:
@@ -511,13 +551,14 @@ def qk_whole_prepare(q, k, v, *, heads: int, kv_heads: int, q_norm=None, k_norm=
 
 
 def paged_attention(q, slab, block_table, tiles, tok_pos, *, kv_heads: int, dv: int, mask: int, mask_size: int, scale: float, softcap: float = 0.0,
-                    sink: bool = False, gate=None, out=None, kernel: str = "general", max_context: int = 0, head_bias=None, weights: int = 0):
+                    sink: bool = False, gate=None, out=None, kernel: str = "general", max_context: int = 0, head_bias=None, weights: int = 0, keep_first: int = 0):
     """``q [T, H, dk]`` (a view with unit inner stride) against ``slab [P, page, kv_heads * (dk + dv)]`` -> ``out [T, H, dv]``
-    (contiguous, the query's dtype).  ``gate [T, H]`` (a view with unit inner stride): logits of a sigmoid output gate.
+    (the query's dtype; given, a view with unit inner stride).  ``gate [T, H]`` (a view with unit inner stride): logits of a sigmoid output gate.
     ``kernel`` and the tile size of ``tiles`` come from ``paged_attention_kernel``.  ``max_context`` (the longest sequence of
     the step, 0 = unknown) lets the tensor-core kernel split the key range over several CTAs when the launch alone would
     leave SMs idle.  ``head_bias`` (fp32 ``[H]``): with ``sink`` the sink's term is ``exp(head_bias[h])`` instead of ``exp(0)``;
-    with ``weights=WEIGHTS_SIGMOID`` there is no softmax, a visible key weighs ``sigmoid(score + head_bias[h])``."""
+    with ``weights=WEIGHTS_SIGMOID`` there is no softmax, a visible key weighs ``sigmoid(score + head_bias[h])``.  ``keep_first``
+    (window mask): the sequence's first positions that stay visible from everywhere after them."""
     _gpu("paged_attention", q, slab, block_table, tiles, tok_pos, gate, out, head_bias)
     if head_bias is not None and (head_bias.dtype != torch.float32 or head_bias.shape != (q.shape[1],) or not head_bias.is_contiguous()):
         raise RuntimeError("paged_attention: head_bias must be float32 [H]")
@@ -530,18 +571,20 @@ def paged_attention(q, slab, block_table, tiles, tok_pos, *, kv_heads: int, dv: 
         raise RuntimeError("paged_attention: gate must be [T, H] of the query's dtype")
     if out is None:
         out = torch.empty((T, H, dv), dtype=q.dtype, device=q.device)
+    elif out.shape != (T, H, dv) or out.dtype != q.dtype or out.stride(2) != 1:
+        raise RuntimeError("paged_attention: out must be [T, H, dv] of the query's dtype with unit inner stride")
     if kernel == "mma":
         if slab.dtype != torch.bfloat16:
             raise RuntimeError("paged_attention: the tensor-core kernel takes a bfloat16 cache")
         lib = library()
-        reach = min(max_context, int(mask_size)) if mask != MASK_CAUSAL else max_context  # keys a query can see at most
+        reach = min(max_context, int(mask_size) + int(keep_first)) if mask != MASK_CAUSAL else max_context  # keys a query can see at most
         group = H // kv_heads
         ctas = tiles.shape[0] * kv_heads * -(-group // min(group, 32))
         splits = attention_splits(ctas, reach, slab.device) if reach else 1
         nbytes = int(lib.tlb_paged_attention_mma_workspace(tiles.shape[0], H, kv_heads, dv, splits))
         ws = torch.empty(nbytes, dtype=torch.uint8, device=slab.device) if nbytes else None
         _check(lib.tlb_paged_attention_mma(_ptr(q), q.stride(0), q.stride(1), _ptr(slab), P, page_size, dk, dv, H, kv_heads, _ptr(block_table),
-                                           block_table.shape[1], _ptr(tiles), tiles.shape[0], _ptr(tok_pos), int(mask), int(mask_size),
+                                           block_table.shape[1], _ptr(tiles), tiles.shape[0], _ptr(tok_pos), int(mask), int(mask_size), int(keep_first),
                                            float(scale), float(softcap or 0.0), int(bool(sink)), _ptr(gate),
                                            gate.stride(0) if gate is not None else 0, _ptr(out), out.stride(0), out.stride(1), splits, _ptr(ws), nbytes,
                                            _ptr(head_bias), int(weights), _stream(q)))
@@ -549,7 +592,7 @@ def paged_attention(q, slab, block_table, tiles, tok_pos, *, kv_heads: int, dv: 
     if kernel != "general":
         raise RuntimeError(f"paged_attention: unknown kernel {kernel!r}")
     _check(library().tlb_paged_attention(_ptr(q), q.stride(0), q.stride(1), _ptr(slab), P, page_size, dk, dv, H, kv_heads, _ptr(block_table),
-                                         block_table.shape[1], _ptr(tiles), tiles.shape[0], _ptr(tok_pos), int(mask), int(mask_size), float(scale),
+                                         block_table.shape[1], _ptr(tiles), tiles.shape[0], _ptr(tok_pos), int(mask), int(mask_size), int(keep_first), float(scale),
                                          float(softcap or 0.0), int(bool(sink)), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(out),
                                          out.stride(0), out.stride(1), _ptr(head_bias), int(weights), _code(q.dtype), _stream(q)))
     return out

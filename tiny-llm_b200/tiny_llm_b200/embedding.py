@@ -25,6 +25,27 @@ class Embedding:
         return linear(x, self.weight)
 
 
+class PairEmbedding:
+    """The start of an fp32 residual stream over a ragged batch: ``table[token] * scale``, plus, with ``pairs [buckets + 1, D]``, a
+    row for the token and the one before it, ``(previous * mul_prev + token * mul_cur) mod buckets``, the last row for a
+    sequence's first token.  The token before comes from the batch or, at the start of a portion, from the request's cache
+    (``RaggedPlan.seq_prev``).  The norms that read the stream first are made in the same launch."""
+
+    def __init__(self, weight: torch.Tensor, scale: float = 1.0, pairs: torch.Tensor | None = None, buckets: int = 0, mul_prev: int = 0, mul_cur: int = 0):
+        self.weight, self.scale = weight.contiguous(), float(scale)
+        self.pairs = None if pairs is None else pairs.contiguous()
+        self.mul_prev, self.mul_cur = int(mul_prev), int(mul_cur)
+        if self.pairs is not None and tuple(self.pairs.shape) != (int(buckets) + 1, self.weight.shape[1]):
+            raise ValueError("pair embedding: the table must be [buckets + 1, width]")
+
+    def __call__(self, plan, eps: float, norm: torch.Tensor, norm2: torch.Tensor | None = None):
+        """-> (x32 [T, D] fp32, the norm times ``norm``, the norm times ``norm2`` or None)."""
+        from extensions_b200.tiny_llm_ext_b200 import blocks
+
+        return blocks.embed_pairs(plan.ids, self.weight, self.scale, pairs=self.pairs, mul_prev=self.mul_prev, mul_cur=self.mul_cur, tok_pos=plan.tok_pos,
+                                  tok_seq=plan.tok_seq, seq_prev=plan.seq_prev, weight=norm, weight2=norm2, eps=eps)
+
+
 class QuantizedEmbedding:
     """Packed table (embedding.py:25-57): readable gather+dequantise, or the
     fused gather kernel when ``use_custom_kernel`` and biases are present."""

@@ -11,6 +11,8 @@ keeps the integers.
 
 from __future__ import annotations
 
+from array import array
+
 import torch
 
 from .kv_cache import TinyKvCache
@@ -86,10 +88,29 @@ class LatentPagedPool(TinyKvPagedPool):
 
 class LatentPagedCache(TinyKvPagedCache):
     """A request's page list (shared by all its layers).  Only the integer side of ``TinyKvPagedCache`` applies:
-    ``append_slots`` / ``rewind`` / ``release`` / ``block_table_host``; rows are written by the append kernel."""
+    ``append_slots`` / ``rewind`` / ``release`` / ``block_table_host``; rows are written by the append kernel.
+    ``tokens`` are the ids the request has run so far (what a model whose embedding looks at the token before reads at the
+    start of the next portion); the step's plan records them."""
 
     def __init__(self, pool: LatentPagedPool):
         super().__init__(pool)
+        self.tokens = array("q")
+
+    def record_tokens(self, ids) -> None:
+        """The ids of the newest ``len(ids)`` slots, after ``append_slots``."""
+        at = self.offset - len(ids)
+        if at > len(self.tokens):  # slots filled by something that is no step: their ids are unknown
+            self.tokens.extend([-1] * (at - len(self.tokens)))
+        del self.tokens[at:]
+        self.tokens.extend(int(t) for t in ids)
+
+    def rewind(self, n: int):
+        super().rewind(n)
+        del self.tokens[self.offset :]
+
+    def release(self):
+        super().release()
+        del self.tokens[:]
 
     def _device(self):
         return self.pool.device

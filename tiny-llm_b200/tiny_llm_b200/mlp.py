@@ -48,12 +48,16 @@ class GatedMLP:
         if act == "clamped_swish" and not self.limit > 0:
             raise ValueError("gated feed-forward: the clamped activation needs a positive limit")
 
-    def __call__(self, h: torch.Tensor, wide: bool = False) -> torch.Tensor:
-        """``wide``: hand the down projection's fp32 accumulator back unrounded (when a norm reads it next)."""
+    def inner(self, h: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
+        """``act(gate h) * (up h)``, the down projection's operand; ``out``: the columns of a wider matrix it goes to."""
         from extensions_b200.tiny_llm_ext_b200 import blocks
 
         first = linear(h, self.w_gate_up) if self.b_gate_up is None else torch.addmm(self.b_gate_up, h, self.w_gate_up.t())
-        return (linear_wide if wide else linear)(blocks.gated_act(first, self.act, self.limit, self.slope), self.w_down)
+        return blocks.gated_act(first, self.act, self.limit, self.slope, out)
+
+    def __call__(self, h: torch.Tensor, wide: bool = False) -> torch.Tensor:
+        """``wide``: hand the down projection's fp32 accumulator back unrounded (when a norm reads it next)."""
+        return (linear_wide if wide else linear)(self.inner(h), self.w_down)
 
 
 class TopKRouter:

@@ -21,6 +21,7 @@ ARCHITECTURES = {
     "Bapovik": ("tiny_llm_b200.bapovik", "BapovikModel"),
     "Senurax": ("tiny_llm_b200.senurax", "SenuraxModel"),
     "Norusun": ("tiny_llm_b200.norusun", "NorusunModel"),
+    "Zalazen": ("tiny_llm_b200.zalazen", "ZalazenModel"),
 }
 
 

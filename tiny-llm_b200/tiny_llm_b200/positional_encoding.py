@@ -2,7 +2,18 @@
 
 from __future__ import annotations
 
+import math
+
 import torch
+
+
+def yarn_ramp(dims: int, base: float, *, factor: float, original: float, fast: float, slow: float) -> tuple:
+    """(factor, lo, hi, gain) of a rotation stretched to ``factor`` times its original context (YaRN): pairs that turn more than
+    ``fast`` times over ``original`` positions keep their frequency, those below ``slow`` turns have it divided by ``factor``,
+    a linear ramp over the pair's number (``lo`` to ``hi``) in between; cos and sin are multiplied by ``gain``."""
+    pair_at = lambda turns: dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+    lo, hi = max(math.floor(pair_at(fast)), 0), min(math.ceil(pair_at(slow)), dims - 1)
+    return (float(factor), float(lo), float(hi), 0.1 * math.log(factor) + 1.0)
 
 
 class RoPE:

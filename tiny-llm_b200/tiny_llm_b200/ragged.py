@@ -4,12 +4,13 @@ A continuous-batching step is a flat list of tokens: a portion of one request's 
 others.  ``RaggedEntry`` names one request's share, ``RaggedPlan`` is what the kernels need, built on the host from the
 requests' page lists and moved to the device as ONE pinned block:
 
-    ids [T] | tok_pos [T] | tok_seq [T] | want_rows [W] | block_table [S, max_pages] | tiles [n, 3] per tile size | seq_info [S, 4]
+    ids [T] | tok_pos [T] | tok_seq [T] | want_rows [W] | block_table [S, max_pages] | tiles [n, 3] per tile size | seq_info [S, 4] | seq_prev [S]
 
 ``tok_pos`` is the position of a token in its sequence, ``tok_seq`` its row in this step's block table, ``tiles`` the
 attention kernels' work lists (runs of at most ``tile`` consecutive tokens of one sequence; one list per tile size
 the model's layers ask for, ``tiles_for(size)``), ``seq_info`` one row per sequence for kernels that walk a sequence's new
-tokens in order (first flat token, token count, position of the first token, the request's recurrent-state slot or -1).
+tokens in order (first flat token, token count, position of the first token, the request's recurrent-state slot or -1),
+``seq_prev`` the token that every sequence ended its last step with (-1: none, or its cache keeps no token history).
 Building the plan also
 does the step's cache bookkeeping: every request's page list grows by its new tokens (pages come from the pool's free
 list first), before anything is launched.
@@ -35,7 +36,7 @@ class RaggedPlan:
     @staticmethod
     def block_ints(tokens: int, wanted: int, seqs: int, max_pages: int, tiles: int) -> int:
         """Number of int32 in a plan's device block (``tiles`` summed over the tile sizes)."""
-        return 3 * tokens + wanted + seqs * max_pages + 3 * tiles + 4 * seqs
+        return 3 * tokens + wanted + seqs * max_pages + 3 * tiles + 5 * seqs
 
     def __init__(self, entries: Sequence[RaggedEntry], device, tile, max_pages: int | None = None, into: torch.Tensor | None = None):
         """``max_pages`` fixes the block table's width (at least what the longest request needs) and ``into`` names a
@@ -82,6 +83,7 @@ class RaggedPlan:
             tile_at[size] = (at, n_tiles[size])
             at += 3 * n_tiles[size]
         info = buf[at : at + 4 * S].reshape(S, 4)
+        prev = buf[at + 4 * S : at + 5 * S]
         tile_rows = {size: [] for size in sizes}
         t = w = 0
         for s, (e, o, start) in enumerate(zip(entries, owners, starts)):
@@ -98,6 +100,8 @@ class RaggedPlan:
                 tile_rows[size] += [(t + first, min(size, n - first), s) for first in range(0, n, size)]
             table[s, : o.num_pages] = o.page_ids
             info[s] = (t, n, start, getattr(o, "state_slot", -1))
+            history = getattr(o, "tokens", None)
+            prev[s] = history[start - 1] if history is not None and 0 < start <= len(history) else -1
             t += n
         for size in sizes:
             start, n = tile_at[size]
@@ -118,24 +122,27 @@ class RaggedPlan:
         self.block_table = dev[3 * T + W : 3 * T + W + S * max_pages].view(S, max_pages)
         self._tiles = {size: dev[start : start + 3 * n].view(n, 3) for size, (start, n) in tile_at.items()}
         self.seq_info = dev[at : at + 4 * S].view(S, 4)
+        self.seq_prev = dev[at + 4 * S : at + 5 * S]
         self.tiles = self._tiles[sizes[0]]
         self.max_context = max(o.offset for o in owners)  # the longest sequence after this step's append
         self.want_counts = [len(x) for x in wants]
         self.starts = starts
         self.max_tokens = max(len(e.tokens) for e in entries)  # the longest entry of the step
         self.owners = owners
-        for o in owners:  # from here on the step runs: what it consumes cannot be taken back from a recurrent state
+        for o, e in zip(owners, entries):  # from here on the step runs: what it consumes cannot be taken back from a recurrent state
+            if hasattr(o, "record_tokens"):
+                o.record_tokens(e.tokens)
             if hasattr(o, "ran_offset"):
                 o.ran_offset = o.offset
 
-    def rope_tables(self, dims: int, base: float, factor: float = 1.0):
+    def rope_tables(self, dims: int, base: float, factor: float = 1.0, ramp: tuple | None = None):
         """(cos, sin) fp32 ``[T, dims // 2]`` of this step's token positions, made once per step and rotation."""
         from extensions_b200.tiny_llm_ext_b200 import blocks
 
-        key = (int(dims), float(base), float(factor))
+        key = (int(dims), float(base), float(factor), ramp)
         tables = self.__dict__.setdefault("_rope_tables", {})
         if key not in tables:
-            tables[key] = blocks.rope_table(self.tok_pos, dims=key[0], base=key[1], factor=key[2])
+            tables[key] = blocks.rope_table(self.tok_pos, dims=key[0], base=key[1], factor=key[2], ramp=key[3])
         return tables[key]
 
     def tiles_for(self, size: int) -> torch.Tensor:
