@@ -562,3 +562,69 @@ def synthetic_norusun(config: dict, seed: int = 0, dtype=torch.bfloat16) -> dict
 
 
 save_norusun = save_voluzen
+
+
+# ---- Zalazen (windowed attention with kept first positions beside a gated feed-forward, pair embedding; zalazen.py) ----
+def zalazen_config(*, width=96, vocab=200, pattern="AdSdAnAd", heads=4, kv_heads=2, dim=16, vdim=24, windows=((24, 3),), rot_dims=8, rot_base=30000.0,
+                   scaling=(4.0, 512, 16.0, 1.0), scale=None, ff=160, embed_scale=5.0, buckets=509, mul_prev=19, mul_cur=11, eps=1e-6) -> dict:
+    """A config.json for a stack spelled by ``pattern``, two letters a layer: the mixer (``A`` attention with keys and values of
+    its own, ``S`` attention over the cache of the nearest ``A`` before it) and the feed-forward (``d`` dense, ``n`` none).
+    ``windows``: (size, kept first positions), taken in turn by the layers; ``scaling``: (factor, original, fast, slow) of the
+    rotation or None; ``buckets`` 0 = no pair table."""
+    if len(pattern) % 2:
+        raise ValueError("the pattern is pairs of letters: mixer, feed-forward")
+    layers, source = [], None
+    for i, (mixer_letter, ff_letter) in enumerate(zip(pattern[0::2], pattern[1::2])):
+        if mixer_letter not in "AS" or ff_letter not in "dn":
+            raise ValueError(f"unknown layer {mixer_letter + ff_letter!r}")
+        size, keep_first = windows[i % len(windows)]
+        rot = {"base": rot_base, "dims": rot_dims}
+        if scaling:
+            rot["scaling"] = dict(zip(("factor", "original", "fast", "slow"), scaling))
+        mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": size, "keep_first": keep_first}, "rot": rot,
+                 "scale": float(scale if scale is not None else dim ** -0.5)}
+        if mixer_letter == "S":
+            if source is None:
+                raise ValueError("an S layer needs an A layer before it")
+            mixer["kv_from"] = source
+        else:
+            source = i
+        layers.append({"type": "attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": ff} if ff_letter == "d" else None})
+    embedding = {"scale": embed_scale}
+    if buckets:
+        embedding["bigram"] = {"buckets": buckets, "mul_prev": mul_prev, "mul_cur": mul_cur}
+    return {"architecture": "Zalazen", "vocab": vocab, "width": width, "norm": {"eps": eps}, "embedding": embedding, "layers": layers}
+
+
+def synthetic_zalazen(config: dict, seed: int = 0, dtype=torch.bfloat16, sharp: float = 1.0) -> dict:
+    """Random tensors for ``config`` under the checkpoint's names (CPU, seeded); ``sharp`` scales the query norms' weights, so
+    that single keys stand out in the softmax."""
+    gen = torch.Generator().manual_seed(seed)
+    D = config["width"]
+
+    def mat(out_dim, in_dim, gain=1.0):
+        return (torch.randn(out_dim, in_dim, generator=gen) * (gain / in_dim**0.5)).to(dtype)
+
+    def vec(n, centre, spread):
+        return (centre + spread * torch.randn(n, generator=gen)).to(dtype)
+
+    tensors = {"embed": (torch.randn(config["vocab"], D, generator=gen) / config["embedding"]["scale"]).to(dtype), "final.norm": vec(D, 1.0, 0.1),
+               "head": mat(config["vocab"], D)}
+    if config["embedding"].get("bigram"):
+        tensors["bigram"] = (0.7 * torch.randn(config["embedding"]["bigram"]["buckets"] + 1, D, generator=gen)).to(dtype)
+    for i, layer in enumerate(config["layers"]):
+        m, p = layer["mixer"], f"l{i}.mix."
+        H, G, dk, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        tensors[f"l{i}.norm1"] = vec(D, 1.0, 0.1)
+        tensors[p + "q"], tensors[p + "q.norm"] = mat(H * dk, D), vec(H * dk, sharp, 0.2 * sharp)
+        if m.get("kv_from") is None:
+            tensors[p + "k"], tensors[p + "v"], tensors[p + "k.norm"] = mat(G * dk, D), mat(G * dv, D), vec(G * dk, 1.0, 0.2)
+        tensors[p + "sink"], tensors[p + "g"], tensors[p + "o"] = vec(H, 0.0, 1.0), mat(H, D, 2.0), mat(D, H * dv, 2.0)
+        if layer.get("mlp"):
+            f = layer["mlp"]["ff"]
+            tensors[f"l{i}.norm2"] = vec(D, 1.0, 0.1)
+            tensors[f"l{i}.mlp.gate"], tensors[f"l{i}.mlp.up"], tensors[f"l{i}.mlp.down"] = mat(f, D, 1.5), mat(f, D), mat(D, f, 1.5)
+    return tensors
+
+
+save_zalazen = save_voluzen
