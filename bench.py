@@ -41,6 +41,9 @@ Numbers on the JSON line (decode):
   --workload norusun  (not a BASELINE config) the Norusun design - residual streams, time-mix linear attention, latent attention with
                       learned sinks, chunked sigmoid attention beside a state-space mixer - at two real-layer sizes beside Senurax of
                       equal size, and its kernels against their rooflines.
+  --workload zalazen  (not a BASELINE config) the Zalazen design - windowed attention with kept first positions, sinks and gates beside a
+                      gated feed-forward, pair embedding - at two real-layer sizes beside Bapovik's attention layers of equal size, and its
+                      kernels against their rooflines.
   --workload bapovik  (not a BASELINE config) the Bapovik design - windowed / chunked attention beside a recurrent mixer, experts,
             bf16 weights - at two sizes beside Voluzen of equal size, and the design's kernels alone against the measured peaks
   cpu_baseline  the reference's CPU path (oracle.model: dense bf16 weights, readable operators) on the
@@ -1652,13 +1655,188 @@ def run_norusun(args) -> None:
                       "steps": steps, "warmup": warmup, "peaks": measured_peaks(), "clocks": clocks, "sizes": results}), flush=True)
 
 
+# ------------------------------------------------------------------ workload: zalazen (windowed attention with kept first positions beside a gated feed-forward; beside Bapovik's attention layers of equal size)
+ZALAZEN_SIZES = {
+    # four layers at sizes that resemble real models of this kind: every second one reads the cache of the layer before it, a dense
+    # feed-forward in each.  The Bapovik arm (the framework's closest model: windowed grouped-query attention with an output gate and
+    # shared caches beside a feed-forward that reads the same stream) has the same width, depth, heads, head sizes, windows and cache
+    # sharing; its ungated feed-forward (one expert that every token takes) has 3/2 of the inner width, so that it has the same number of weights.
+    "w1024": dict(width=1024, vocab=32768, pattern="AdSdAdSd", heads=8, kv_heads=2, dim=128, vdim=128, windows=((512, 4),), rot_dims=64, rot_base=100000.0,
+                  scaling=(4.0, 4096, 32.0, 1.0), ff=2816, buckets=65521),
+    "w2048": dict(width=2048, vocab=32768, pattern="AdSdAdSd", heads=16, kv_heads=4, dim=128, vdim=128, windows=((1024, 16),), rot_dims=64, rot_base=100000.0,
+                  scaling=(4.0, 4096, 32.0, 1.0), ff=5632, buckets=65521),
+}
+
+
+def _zalazen_kernels(cfg: dict, device, prompt: int, batch: int, context: int) -> dict:
+    """The kernels the design added or extended, alone at this size, CUDA-event timed after warm-up, each against the roofline
+    of its kind (measured copy bandwidth for row kernels, measured cuBLAS bf16 burst for contractions), the like kernel of the
+    framework's other models beside it where there is one; between repetitions a 256 MB buffer is rewritten to flush L2."""
+    from extensions_b200.tiny_llm_ext_b200 import blocks
+    from tiny_llm_b200.basics import linear_wide
+    from tiny_llm_b200.paged_attention import JoinedProjection
+    from tiny_llm_b200.positional_encoding import yarn_ramp
+
+    peaks = measured_peaks()
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=device)
+    bf = torch.bfloat16
+
+    def timed(fn, reps=7):
+        for _ in range(3):
+            fn()
+        best = []
+        for _ in range(reps):
+            flush.fill_(1)
+            best.append(cuda_time_ms(fn))
+        return statistics.median(best)
+
+    def stream(nbytes, ms, **more):
+        return dict(more, ms=round(ms, 4), gbs=round(nbytes / ms / 1e6, 1), of_measured_hbm=round(nbytes / ms / 1e6 / peaks["hbm_gbs"], 4))
+
+    def math(flops, ms, **more):
+        return dict(more, ms=round(ms, 4), tflops=round(flops / ms / 1e9, 1), of_measured_bf16_burst=round(flops / ms / 1e9 / peaks["bf16_tflops"], 4))
+
+    out = {}
+    D, V, rows, eps = cfg["width"], cfg["vocab"], 32768, 1e-6
+    pos, seq = torch.arange(rows, dtype=torch.int32, device=device), torch.zeros(rows, dtype=torch.int32, device=device)
+    w1, w2 = torch.ones(D, device=device).to(bf), torch.ones(D, device=device).to(bf)
+    ids = torch.randint(0, V, (rows,), dtype=torch.int32, device=device)
+    table, pairs = torch.randn((V, D), device=device).to(bf), torch.randn((cfg["buckets"] + 1, D), device=device).to(bf)
+    prev = torch.zeros(1, dtype=torch.int32, device=device)
+    ms = timed(lambda: blocks.embed_pairs(ids, table, 4.0, pairs=pairs, mul_prev=31337, mul_cur=7919, tok_pos=pos, tok_seq=seq, seq_prev=prev, weight=w1, weight2=w2, eps=eps))
+    out["embedding_pair_two_norms"] = stream(rows * D * (2 + 2 + 4 + 2 + 2), ms, rows=rows)
+    ms = timed(lambda: blocks.embed_rows(ids, table))
+    out["like_embed_rows"] = stream(rows * D * (2 + 4 + 2), ms, rows=rows)
+    del table, pairs
+    x, y = torch.randn((rows, D), device=device), torch.randn((rows, D), device=device)
+    ms = timed(lambda: blocks.add_norm(x, y, None, w1, eps, w2))
+    out["residual_two_norms"] = stream(rows * D * (4 + 4 + 4 + 2 + 2), ms, rows=rows)
+    ms = timed(lambda: blocks.add_norm(x, y, y, w1, eps))
+    out["like_add_norm"] = stream(rows * D * (4 + 4 + 4 + 4 + 2), ms, rows=rows)
+    few, fy = x[:batch], y[:batch]
+    ms = timed(lambda: blocks.add_norm(few, fy, None, w1, eps, w2))
+    out["residual_two_norms_decode"] = stream(batch * D * (4 + 4 + 4 + 2 + 2), ms, batch=batch)
+
+    H, G, dk, dv, rot = cfg["heads"], cfg["kv_heads"], cfg["dim"], cfg["vdim"], cfg["rot_dims"]
+    base, page = cfg["rot_base"], 64
+    ramp = yarn_ramp(rot, base, **dict(zip(("factor", "original", "fast", "slow"), cfg["scaling"])))
+    ms = timed(lambda: blocks.rope_table(pos, dims=rot, base=base, ramp=ramp))
+    out["rotation_table"] = stream(rows * rot * 4, ms, rows=rows, note="once per step, all layers share it")
+    angles = blocks.rope_table(pos, dims=rot, base=base, ramp=ramp)
+    width = H * dk + G * (dk + dv) + H
+    wide = torch.randn((rows, width + -width % 8), device=device).to(bf)      # q | k | v | gate, as the layer's product leaves them
+    q, k, v = wide[:, : H * dk], wide[:, H * dk : (H + G) * dk], wide[:, (H + G) * dk : (H + G) * dk + G * dv]
+    qw, kw = torch.ones(H * dk, device=device).to(bf), torch.ones(G * dk, device=device).to(bf)
+    slab = torch.empty((rows // page, page, G * (dk + dv)), dtype=bf, device=device)
+    block_table = torch.arange(rows // page, dtype=torch.int32, device=device).view(1, -1)
+
+    def prepare(n, own, rope=angles, dims=rot):
+        blocks.qk_whole_prepare(q[:n], k[:n] if own else None, v[:n] if own else None, heads=H, kv_heads=G, q_norm=qw, k_norm=kw if own else None, eps=eps,
+                                rot_dims=dims, base=base, tok_pos=pos[:n], tok_seq=seq[:n], block_table=block_table, slab=slab if own else None,
+                                rope=(rope[0][:n], rope[1][:n]))
+
+    ms = timed(lambda: prepare(rows, True))
+    out["whole_norm_rotation_cache_store"] = stream(rows * (H * dk + G * (dk + dv)) * 2 * 2, ms, rows=rows)
+    ms = timed(lambda: prepare(rows, False))
+    out["whole_norm_rotation_queries"] = stream(rows * H * dk * 2 * 2, ms, rows=rows)
+    ms = timed(lambda: prepare(batch, True))
+    out["whole_norm_rotation_cache_store_decode"] = stream(batch * (H * dk + G * (dk + dv)) * 2 * 2, ms, batch=batch)
+    full = blocks.rope_table(pos, dims=dk, base=base)
+    ms = timed(lambda: prepare(rows, True, full, dk))
+    out["like_whole_norm_full_rotation"] = stream(rows * (H * dk + G * (dk + dv)) * 2 * 2, ms, rows=rows)
+    del wide, q, k, v, slab
+
+    window, keep = cfg["windows"][0]
+    kernel, tile = blocks.paged_attention_kernel(bf, H, G, dk, dv, page)
+    sink = torch.randn(H, device=device)
+
+    def attention(tokens_per_seq, seqs, ctx, plain=False):
+        pages_per = -(-ctx // page)
+        slab = torch.randn((seqs * pages_per, page, G * (dk + dv)), dtype=torch.float32, device=device).to(bf)
+        table = torch.arange(seqs * pages_per, dtype=torch.int32, device=device).view(seqs, pages_per)
+        T = tokens_per_seq * seqs
+        tok = torch.cat([torch.arange(ctx - tokens_per_seq, ctx, dtype=torch.int32) for _ in range(seqs)]).to(device)
+        tiles = torch.tensor([(s * tokens_per_seq + f, min(tile, tokens_per_seq - f), s) for s in range(seqs) for f in range(0, tokens_per_seq, tile)],
+                             dtype=torch.int32, device=device)
+        q, gate = torch.randn((T, H, dk), device=device).to(bf), torch.randn((T, H), device=device).to(bf)
+        o = torch.empty((T, H * dv + cfg["ff"]), dtype=bf, device=device)[:, : H * dv].unflatten(1, (H, dv))
+        more = {} if plain else dict(keep_first=keep, sink=True, head_bias=sink)
+        return timed(lambda: blocks.paged_attention(q, slab, table, tiles, tok, kv_heads=G, dv=dv, mask=blocks.MASK_WINDOW, mask_size=window, scale=dk ** -0.5,
+                                                    gate=gate, out=o, kernel=kernel, max_context=ctx, **more))
+
+    for name, plain in (("window_kept_sink_attention", False), ("like_window_attention", True)):
+        kept = 0 if plain else keep
+        ms = attention(prompt, 1, prompt, plain)
+        seen = sum(min(p + 1, window) + max(0, min(kept, p + 1 - window)) for p in range(prompt))
+        out[name + "_prefill"] = math(2.0 * H * (dk + dv) * seen, ms, kernel=kernel, tokens=prompt, window=window, keep_first=kept)
+        ms = attention(1, batch, context, plain)
+        seen = min(context, window) + max(0, min(kept, context - window))
+        out[name + "_decode"] = stream(batch * seen * G * (dk + dv) * 2, ms, kernel=kernel, batch=batch, context=context)
+    ff = cfg["ff"]
+    for n, name in ((rows // 4, "gated_silu"), (batch, "gated_silu_decode")):
+        gu, dst = torch.randn((n, 2 * ff), device=device).to(bf), torch.empty((n, H * dv + ff), dtype=bf, device=device)
+        ms = timed(lambda: blocks.gated_act(gu, blocks.ACT_SILU, out=dst[:, H * dv :]))
+        out[name] = stream(n * ff * 3 * 2, ms, rows=n, note="into its columns of the joined product's operand")
+    gu = torch.randn((rows // 4, 2 * ff), device=device).to(bf)
+    ms = timed(lambda: blocks.gated_act(gu, blocks.ACT_SILU))
+    out["like_gated_silu"] = stream(rows // 4 * ff * 3 * 2, ms, rows=rows // 4)
+    w_o, w_down = (torch.randn((D, H * dv), device=device) / (H * dv) ** 0.5).to(bf), (torch.randn((D, ff), device=device) / ff**0.5).to(bf)
+    joined = JoinedProjection([("o", w_o), ("down", w_down)])
+    for n, name in ((prompt, "prefill"), (batch, "decode")):
+        operand, part = joined.operand(n)
+        operand.normal_()
+        a, b = part["o"].contiguous(), part["down"].contiguous()
+        ms = timed(lambda: joined(operand))
+        out["joined_product_" + name] = math(2.0 * n * D * (H * dv + ff), ms, tokens=n, note="library product; weights %.1f MB" % (joined.weight.numel() * 2 / 1e6))
+        ms = timed(lambda: (linear_wide(a, w_o), linear_wide(b, w_down)))
+        out["like_two_products_" + name] = math(2.0 * n * D * (H * dv + ff), ms, tokens=n, note="without the addition that would follow")
+    return out
+
+
+def run_zalazen(args) -> None:
+    """Prefill and decode throughput of the Zalazen design at ZALAZEN_SIZES beside Bapovik (the framework's closest model) of
+    equal size, through the same ragged step; and the design's kernels against their rooflines.  One JSON line; random
+    weights, random prompts."""
+    from tiny_llm_b200.models import model_class
+    from tiny_llm_b200.synthetic import bapovik_config, synthetic_bapovik, synthetic_zalazen, zalazen_config
+
+    device = torch.device("cuda:0")
+    prompt, batch, context, steps = args.prompt_len or 2048, 16, 1024, max(args.steps or 16, 4)
+    warmup = max(args.warmup, 3)
+    sampler = ClockSampler(0)
+    sampler.start()
+    results = []
+    for name, size in ZALAZEN_SIZES.items():
+        config = zalazen_config(**size)
+        model = model_class("Zalazen").from_checkpoint(config, synthetic_zalazen(config, seed=0), device=device, dtype=torch.bfloat16)
+        entry = {"size": name, "config": dict(size), "prompt_tokens": prompt, "decode_batch": batch, "decode_context": context,
+                 "zalazen": _measure_ragged(model, size["vocab"], prompt, batch, context, steps, warmup)}
+        entry["zalazen_batch1"] = _measure_ragged(model, size["vocab"], prompt, 1, context, steps, warmup)
+        entry["kernels"] = _zalazen_kernels(size, device, prompt, batch, context)
+        del model
+        torch.cuda.empty_cache()
+        bsize = dict(width=size["width"], vocab=size["vocab"], pattern="ASAS", heads=size["heads"], kv_heads=size["kv_heads"], dim=size["dim"], vdim=size["vdim"],
+                     window=size["windows"][0][0], experts=1, top=1, expert_ff=size["ff"] * 3 // 2)
+        bconfig = bapovik_config(**bsize)
+        other = model_class("Bapovik").from_checkpoint(bconfig, synthetic_bapovik(bconfig, seed=0), device=device, dtype=torch.bfloat16)
+        entry["bapovik_equal_size"] = dict(_measure_ragged(other, size["vocab"], prompt, batch, context, steps, warmup), config=bsize)
+        entry["bapovik_equal_size_batch1"] = _measure_ragged(other, size["vocab"], prompt, 1, context, steps, warmup)
+        del other
+        torch.cuda.empty_cache()
+        results.append(entry)
+    clocks = sampler.stop()
+    print(json.dumps({"workload": "zalazen", "metric": "Zalazen prefill / decode tok/s beside Bapovik of equal size", "unit": UNIT, "n_gpus": 1,
+                      "dtype": "bf16 (unquantised weights in both)", "data": "synthetic (random weights, random prompts)",
+                      "steps": steps, "warmup": warmup, "peaks": measured_peaks(), "clocks": clocks, "sizes": results}), flush=True)
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=None)
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--impl", choices=["ours", "reference"], default="ours")
-    ap.add_argument("--workload", choices=sorted(METRICS) + ["voluzen", "bapovik", "senurax", "norusun"], default="decode")
+    ap.add_argument("--workload", choices=sorted(METRICS) + ["voluzen", "bapovik", "senurax", "norusun", "zalazen"], default="decode")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-extra", action="store_true", help="skip the sweeps / secondary measurements under `extra`")
     ap.add_argument("--requests", type=int, default=0, help="serve/serve8k: total requests over all ranks")
@@ -1676,6 +1854,8 @@ def main() -> None:
         run_senurax(args)
     elif args.workload == "norusun":
         run_norusun(args)
+    elif args.workload == "zalazen":
+        run_zalazen(args)
     elif args.impl == "reference":
         run_reference(args)
     elif args.workload == "decode":

@@ -143,6 +143,16 @@ int tlb_paged_attention_mma(const void *q, long long q_token, long long q_head, 
 /* splits > 1 cuts every tile's key range over that many CTAs (few query rows, long key ranges) and a second launch merges the
  * partial sums; workspace: tlb_paged_attention_mma_workspace(...) bytes, no initialisation needed. */
 size_t tlb_paged_attention_mma_workspace(int num_tiles, int heads, int kv_heads, int dv, int splits);
+/* The same with the softmax in registers and 64-key tiles, in two forms: 64 query rows per CTA (split_keys 0: prompt portions)
+ * or 16 rows whose keys the warps share (split_keys 1: single tokens; up to 16 query heads per key/value head).  tile_tokens =
+ * tlb_paged_attention_flash_tile_tokens(heads, kv_heads, split_keys), 0 = the form does not serve these head counts.  splits
+ * (1 to 8): CTAs of one cluster that share a tile's key range and combine their sums through distributed shared memory. */
+int tlb_paged_attention_flash_tile_tokens(int heads, int kv_heads, int split_keys);
+int tlb_paged_attention_flash_supported(int dk, int dv, int kv_heads, int page_size);
+int tlb_paged_attention_flash(const void *q, long long q_token, long long q_head, const void *slab, int num_pages, int page_size, int dk, int dv, int heads,
+                              int kv_heads, const int32_t *block_table, int max_pages, const int32_t *tiles, int num_tiles, const int32_t *tok_pos,
+                              int mask, int mask_size, int keep_first, float scale, float softcap, int sink, const void *gate, long long g_token, void *out,
+                              long long o_token, long long o_head, int split_keys, int splits, const float *head_bias, int weights, void *stream);
 /* Before that attention: per-head RMS norm (plain weight [dk]) of the queries in place (q_norm != NULL) and of the keys
  * (k_norm != NULL), and the token's keys and values stored at its slot of the cache (k != NULL). */
 int tlb_kv_prepare(void *q, long long q_token, long long q_head, int heads, const void *q_norm, const void *k, long long k_token, long long k_head,

@@ -288,7 +288,7 @@ def test_rotated_attention_finds_one_key_far_away_and_at_page_borders(dev, kerne
         for sizes in ([S], [S - 1, 1], [33, 31, S - 64 - 2, 2]):
             lo, rows = 0, []
             for n in sizes:
-                plan = RaggedPlan([RaggedEntry(list(range(n)), [cache], want=range(n))], dev, [att.tile_tokens])
+                plan = RaggedPlan([RaggedEntry(list(range(n)), [cache], want=range(n))], dev, att.tile_sizes)
                 rows.append(att(q[lo : lo + n].reshape(n, -1).to(dev).clone(), k[lo : lo + n].reshape(n, -1).to(dev).clone(), v[lo : lo + n].reshape(n, -1).to(dev),
                                 None, plan, pool.slabs[0]))
                 lo += n

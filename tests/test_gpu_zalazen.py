@@ -184,6 +184,11 @@ def tiles_for(dev, first, count, size):
 WINDOWS = [(24, 0), (24, 1), (24, 5), (31, 32), (20, 33), (64, 64), (70, 3), (1, 4), (1, 0), (33, 100), (5, 700), (1000, 2)]
 
 
+def attention_choices(dtype, heads, kv_heads, dk, dv):
+    """(kernel, most tokens of a work-list entry) of every kernel that serves these sizes."""
+    return [blocks.paged_attention_kernel(dtype, heads, kv_heads, dk, dv, 64)] + list(blocks.paged_attention_flash_forms(dtype, heads, kv_heads, dk, dv, 64).items())
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("heads,kv_heads,dk,dv", [(4, 2, 16, 24), (6, 2, 12, 10), (40, 1, 8, 16)])
 @pytest.mark.parametrize("size,keep", WINDOWS)
@@ -207,29 +212,29 @@ def test_window_with_kept_first_positions_and_sinks_at_every_edge(dev, dtype, he
     plain = lambda keep: O.sink_window_attention(q.double(), k.double(), v.double(), sink.double(), scale=scale, size=size, keep_first=keep)
     want = plain(keep) * torch.sigmoid(gate.double())[:, :, None]
     slab, table = fill_cache(dev, torch.cat([k.reshape(T, -1), v.reshape(T, -1)], dim=1), 64, dtype)
-    kernel, tile = blocks.paged_attention_kernel(dtype, heads, kv_heads, dk, dv, 64)
     pos = torch.arange(T, dtype=torch.int32, device=dev)
     qd, gd, tol = q.to(dev), gate.to(dev), 2e-5 if dtype == torch.float32 else 3e-2
 
-    def run(lo, hi, keep=keep, sink_on=True, split=True):
-        wide = torch.full((hi - lo, heads * dv + 5), 3.0, dtype=dtype, device=dev)
-        blocks.paged_attention(qd[lo:hi], slab, table, tiles_for(dev, 0, hi - lo, tile), pos[lo:hi], kv_heads=kv_heads, dv=dv, mask=blocks.MASK_WINDOW,
-                               mask_size=size, keep_first=keep, scale=scale, sink=sink_on, head_bias=sink.to(dev) if sink_on else None, gate=gd[lo:hi],
-                               kernel=kernel, max_context=hi if split else 0, out=wide[:, : heads * dv].unflatten(1, (heads, dv)))
-        assert float(wide[:, -5:].float().sub(3.0).abs().max()) == 0.0
-        return wide[:, : heads * dv].unflatten(1, (heads, dv))
+    for kernel, tile in attention_choices(dtype, heads, kv_heads, dk, dv):
+        def run(lo, hi, keep=keep, sink_on=True, split=True):
+            wide = torch.full((hi - lo, heads * dv + 5), 3.0, dtype=dtype, device=dev)
+            blocks.paged_attention(qd[lo:hi], slab, table, tiles_for(dev, 0, hi - lo, tile), pos[lo:hi], kv_heads=kv_heads, dv=dv, mask=blocks.MASK_WINDOW,
+                                   mask_size=size, keep_first=keep, scale=scale, sink=sink_on, head_bias=sink.to(dev) if sink_on else None, gate=gd[lo:hi],
+                                   kernel=kernel, max_context=hi if split else 0, out=wide[:, : heads * dv].unflatten(1, (heads, dv)))
+            assert float(wide[:, -5:].float().sub(3.0).abs().max()) == 0.0
+            return wide[:, : heads * dv].unflatten(1, (heads, dv))
 
-    whole = run(0, T)
-    close(whole, want, tol)
-    cut = torch.cat([run(lo, min(lo + 170, T), split=False) for lo in range(0, T, 170)])
-    assert torch.equal(cut, run(0, T, split=False))                      # where a prompt was cut leaves no trace (one CTA per tile)
-    close(torch.cat([run(p, p + 1) for p in list(range(0, 70, 3)) + list(range(380, T))]), torch.cat([want[0:70:3], want[380:]]), tol)
-    close(torch.cat([run(p, p + 2) for p in range(180, 240, 2)]), want[180:240], tol)
-    if heads >= 6:                                                       # the construction shows what it is meant to show
-        assert (run(0, T, sink_on=False).double().cpu() - want).abs().max() > 0.05
-    if 0 < keep < 300 and size < 200 and (heads >= 4 or keep == 1):
-        assert (plain(keep - 1) * torch.sigmoid(gate.double())[:, :, None] - want).abs().max() > 0.05
-        assert (run(0, T, keep=keep - 1).double().cpu() - want).abs().max() > 0.05
+        whole = run(0, T)
+        close(whole, want, tol)
+        cut = torch.cat([run(lo, min(lo + 170, T), split=False) for lo in range(0, T, 170)])
+        assert torch.equal(cut, run(0, T, split=False))                      # where a prompt was cut leaves no trace (one CTA per tile)
+        close(torch.cat([run(p, p + 1) for p in list(range(0, 70, 3)) + list(range(380, T))]), torch.cat([want[0:70:3], want[380:]]), tol)
+        close(torch.cat([run(p, p + 2) for p in range(180, 240, 2)]), want[180:240], tol)
+        if heads >= 6:                                                       # the construction shows what it is meant to show
+            assert (run(0, T, sink_on=False).double().cpu() - want).abs().max() > 0.05
+        if 0 < keep < 300 and size < 200 and (heads >= 4 or keep == 1):
+            assert (plain(keep - 1) * torch.sigmoid(gate.double())[:, :, None] - want).abs().max() > 0.05
+            assert (run(0, T, keep=keep - 1).double().cpu() - want).abs().max() > 0.05
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -253,8 +258,9 @@ def test_a_kept_position_thousands_of_keys_back(dev, dtype):
     slab, table = fill_cache(dev, rows, 64, dtype)
     dead = [p for p in range(-(-T // 64)) if p * 64 + 63 < T - size - 64 and p * 64 >= 64]
     slab[table[0, dead].long()] = float("nan")
-    kernel, tile = blocks.paged_attention_kernel(dtype, heads, kv_heads, dk, dv, 64)
-    for max_context in (0, T):                                           # one CTA per tile, or the key range split over several
+    choices = attention_choices(dtype, heads, kv_heads, dk, dv)
+    assert len(choices) == (1 if dtype == torch.float32 else 3)
+    for (kernel, tile), max_context in [(c, m) for c in choices for m in (0, T)]:   # one CTA per tile, or the key range split over several
         out = blocks.paged_attention(q.to(dtype).to(dev), slab, table, tiles_for(dev, 0, 1, tile), ints(dev, [T - 1]), kv_heads=kv_heads, dv=dv,
                                      mask=blocks.MASK_WINDOW, mask_size=size, keep_first=keep, scale=0.25, sink=True, head_bias=sink.to(dev), kernel=kernel,
                                      max_context=max_context)

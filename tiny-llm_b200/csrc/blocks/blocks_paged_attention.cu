@@ -315,6 +315,98 @@ qk_whole_prepare_kernel(T *q, long long q_token, int heads, const T *__restrict_
     }
 }
 
+// The same step in 16-byte accesses, for bf16 rows whose parts start at 16-byte boundaries and whose rotation is tabulated: a CTA
+// per token, eight adjacent columns per thread - first the queries' columns, then the keys', then the values' - all loads in
+// flight at once, the partner columns of a rotated chunk (rot_dims / 2 further or nearer, a multiple of 8; or the neighbour
+// inside the chunk) read by the thread itself.  A token's numbers depend on nothing but its own row.
+__device__ __forceinline__ void qk_unpack8(uint4 u, float (&x)[8]) {
+    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        float2 f = tl::unpack2<bf16>(w[e]);
+        x[2 * e] = f.x, x[2 * e + 1] = f.y;
+    }
+}
+
+template <bool INTERLEAVED>
+__global__ void qk_whole_prepare_wide_kernel(bf16 *q, long long q_token, int heads, const bf16 *__restrict__ q_norm, const bf16 *__restrict__ k,
+                                             long long k_token, const bf16 *__restrict__ v, long long v_token, int kv_heads, int dk, int dv,
+                                             const bf16 *__restrict__ k_norm, float eps, int rot_dims, const int32_t *__restrict__ tok_pos,
+                                             const int32_t *__restrict__ tok_seq, const int32_t *__restrict__ block_table, int max_pages, int num_pages,
+                                             int page_size, bf16 *__restrict__ slab, const float *__restrict__ rope_cos, const float *__restrict__ rope_sin) {
+    __shared__ float partial[2][32];
+    const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int q_chunks = heads * dk / 8, k_chunks = k ? kv_heads * dk / 8 : 0, v_chunks = k ? kv_heads * dv / 8 : 0;
+    bf16 *dst = nullptr;
+    if (k != nullptr) {
+        const int pos = tok_pos[t];
+        const int page = block_table[(size_t)tok_seq[t] * max_pages + pos / page_size];
+        if (page >= 0 && page < num_pages) dst = slab + ((size_t)page * page_size + pos % page_size) * ((size_t)kv_heads * (dk + dv));
+    }
+    int c = threadIdx.x;
+    const bool is_q = c < q_chunks, is_k = !is_q && c < q_chunks + k_chunks, is_v = !is_q && !is_k && c < q_chunks + k_chunks + v_chunks;
+    if (is_k) c -= q_chunks;
+    if (is_v) c -= q_chunks + k_chunks;
+    float x[8], y[8], g[8], gy[8], cs[8], sn[8];
+    bool turned = false, low = false;
+    if (is_v) {
+        if (dst) *reinterpret_cast<uint4 *>(dst + (size_t)kv_heads * dk + c * 8) = *reinterpret_cast<const uint4 *>(v + (size_t)t * v_token + c * 8);
+    }
+    float sq = 0.f;
+    const bf16 *src = is_q ? q + (size_t)t * q_token : k + (is_k ? (size_t)t * k_token : 0), *w = is_q ? q_norm : k_norm;
+    if (is_q || is_k) {
+        const int e = c * 8 % dk, half = rot_dims / 2;  // the chunk's place in its head
+        qk_unpack8(*reinterpret_cast<const uint4 *>(src + c * 8), x);
+        if (w) qk_unpack8(*reinterpret_cast<const uint4 *>(w + c * 8), g);
+        turned = e < rot_dims;
+        if (turned) {
+            const int i0 = INTERLEAVED ? e / 2 : (e < half ? e : e - half);
+            low = e < half;
+            const float4 *cp = reinterpret_cast<const float4 *>(rope_cos + (size_t)t * half + i0), *sp = reinterpret_cast<const float4 *>(rope_sin + (size_t)t * half + i0);
+            const float4 c0 = cp[0], s0 = sp[0];
+            cs[0] = c0.x, cs[1] = c0.y, cs[2] = c0.z, cs[3] = c0.w, sn[0] = s0.x, sn[1] = s0.y, sn[2] = s0.z, sn[3] = s0.w;
+            if (!INTERLEAVED) {
+                const float4 c1 = cp[1], s1 = sp[1];
+                cs[4] = c1.x, cs[5] = c1.y, cs[6] = c1.z, cs[7] = c1.w, sn[4] = s1.x, sn[5] = s1.y, sn[6] = s1.z, sn[7] = s1.w;
+                const int other = c * 8 + (low ? half : -half);
+                qk_unpack8(*reinterpret_cast<const uint4 *>(src + other), y);
+                if (w) qk_unpack8(*reinterpret_cast<const uint4 *>(w + other), gy);
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) sq = fmaf(x[j], x[j], sq);
+    }
+    const float a = warp_sum(is_q ? sq : 0.f), b = warp_sum(is_k ? sq : 0.f);
+    if (lane == 0) partial[0][warp] = a, partial[1][warp] = b;
+    __syncthreads();  // also: every read of the row is done before its queries change
+    if (!is_q && !is_k) return;
+    float total = 0.f;
+    for (int i = 0; i < (int)(blockDim.x >> 5); ++i) total += partial[is_q ? 0 : 1][i];
+    const float inv = w ? 1.0f / sqrtf(total / (float)((is_q ? heads : kv_heads) * dk) + eps) : 1.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) x[j] = x[j] * inv * (w ? g[j] : 1.f);
+    if (turned) {
+        if (INTERLEAVED) {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const float u = x[2 * j], z = x[2 * j + 1];
+                x[2 * j] = u * cs[j] - z * sn[j], x[2 * j + 1] = z * cs[j] + u * sn[j];
+            }
+        } else {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                const float z = y[j] * inv * (w ? gy[j] : 1.f);
+                x[j] = low ? x[j] * cs[j] - z * sn[j] : x[j] * cs[j] + z * sn[j];
+            }
+        }
+    }
+    bf16 *out = is_q ? q + (size_t)t * q_token : dst;
+    if (out == nullptr) return;
+    uint4 r;
+    r.x = tl::pack2<bf16>(x[0], x[1]), r.y = tl::pack2<bf16>(x[2], x[3]), r.z = tl::pack2<bf16>(x[4], x[5]), r.w = tl::pack2<bf16>(x[6], x[7]);
+    *reinterpret_cast<uint4 *>(out + c * 8) = r;
+}
+
 template <typename T, int VL>
 static int pa_launch(const void *q, long long q_token, long long q_head, const void *slab, int num_pages, int page_size, int dk, int dv, int heads,
                      int kv_heads, const int32_t *block_table, int max_pages, const int32_t *tiles, int num_tiles, const int32_t *tok_pos, int mask,
@@ -402,6 +494,19 @@ int tlb_qk_whole_prepare(void *q, long long q_token, int heads, const void *q_no
     if (k && (!v || !slab || !tok_seq || !block_table || kv_heads <= 0 || dv <= 0 || page_size <= 0 || max_pages <= 0))
         return tl::fail(TL_EINVAL, "qk_whole_prepare: bad cache argument");
     if (!k) kv_heads = 0;
+    // 16-byte accesses where every part's columns allow them (a property of the sizes and the layout, not of the step)
+    const int chunks = heads * dk / 8 + (k ? kv_heads * (dk + dv) / 8 : 0);
+    const auto eights = [](const void *p, long long stride) { return tl::aligned16(p) && stride % 8 == 0; };
+    if (dtype == TL_BF16 && dk % 8 == 0 && (!k || dv % 8 == 0) && rot_dims % (interleaved ? 8 : 16) == 0 && (rot_dims == 0 || (rope_cos && tl::aligned16(rope_cos) && tl::aligned16(rope_sin))) &&
+        chunks <= 1024 && eights(q, q_token) && (!k || (eights(k, k_token) && eights(v, v_token) && tl::aligned16(slab))) && (!q_norm || tl::aligned16(q_norm)) &&
+        (!k_norm || tl::aligned16(k_norm))) {
+        auto kernel = interleaved ? qk_whole_prepare_wide_kernel<true> : qk_whole_prepare_wide_kernel<false>;
+        kernel<<<tokens, ceil_div(chunks, 32) * 32, 0, as_stream(stream)>>>((bf16 *)q, q_token, heads, (const bf16 *)q_norm, (const bf16 *)k, k_token, (const bf16 *)v,
+                                                                            v_token, kv_heads, dk, dv, (const bf16 *)k_norm, eps, rot_dims, tok_pos, tok_seq, block_table,
+                                                                            max_pages, num_pages, page_size, (bf16 *)slab, rope_cos, rope_sin);
+        TL_LAUNCH_CHECK("qk_whole_prepare_wide");
+        return TL_OK;
+    }
     const size_t per_token = ((size_t)(heads > kv_heads ? heads : kv_heads) * dk + rot_dims) * sizeof(float);
     if (per_token > 200 * 1024) return tl::fail(TL_EINVAL, "qk_whole_prepare: a projection of %d entries does not fit in shared memory", heads * dk);
     // a warp per token when there are tokens enough to fill the GPU that way and eight rows fit in shared memory, else a CTA per token

@@ -48,6 +48,7 @@ BLOCKS_SOURCES = [
     "blocks/blocks_moe.cu",
     "blocks/blocks_paged_attention.cu",
     "blocks/blocks_paged_attention_mma.cu",
+    "blocks/blocks_paged_attention_flash.cu",
     "blocks/blocks_linear_attention.cu",
     "blocks/blocks_delta_rule.cu",
     "blocks/blocks_streams.cu",

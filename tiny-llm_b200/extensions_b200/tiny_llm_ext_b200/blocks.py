@@ -53,6 +53,10 @@ _SIGNATURES = {
     "tlb_paged_attention_mma": (_I, [_VP, _LL, _LL, _VP, _I, _I, _I, _I, _I, _I, _VP, _I, _VP, _I, _VP, _I, _I, _I, _F, _F, _I, _VP, _LL, _VP, _LL, _LL, _I, _VP,
                                      ctypes.c_size_t, _VP, _I, _VP]),
     "tlb_paged_attention_mma_workspace": (ctypes.c_size_t, [_I, _I, _I, _I, _I]),
+    "tlb_paged_attention_flash_tile_tokens": (_I, [_I, _I, _I]),
+    "tlb_paged_attention_flash_supported": (_I, [_I, _I, _I, _I]),
+    "tlb_paged_attention_flash": (_I, [_VP, _LL, _LL, _VP, _I, _I, _I, _I, _I, _I, _VP, _I, _VP, _I, _VP, _I, _I, _I, _F, _F, _I, _VP, _LL, _VP, _LL, _LL, _I, _I,
+                                       _VP, _I, _VP]),
     "tlb_kv_prepare": (_I, [_VP, _LL, _LL, _I, _VP, _VP, _LL, _LL, _VP, _LL, _LL, _I, _I, _I, _VP, _F, _VP, _VP, _VP, _I, _I, _I, _VP, _I, _I, _VP]),
     "tlb_qk_whole_prepare": (_I, [_VP, _LL, _I, _VP, _VP, _LL, _VP, _LL, _I, _I, _I, _VP, _F, _I, _I, _D, _VP, _VP, _VP, _I, _I, _I, _VP, _VP, _VP, _I, _I, _VP]),
     "tlb_decay_scan_workspace": (ctypes.c_size_t, [_I, _I, _I, _I, _I]),
@@ -317,13 +321,17 @@ def attention_kernel(dtype, heads: int, rank: int, rot: int, page_size: int) -> 
 _SM_COUNT: dict = {}
 
 
-def attention_splits(num_ctas: int, max_context: int, device) -> int:
-    """Into how many CTAs to cut every tile's key range: 1 while the launch fills the GPU by itself, else enough to give
-    every SM a CTA, each with at least two 64-key tiles."""
+def sm_count(device) -> int:
     key = torch.device(device)
     if key not in _SM_COUNT:
         _SM_COUNT[key] = torch.cuda.get_device_properties(key).multi_processor_count
-    sms = _SM_COUNT[key]
+    return _SM_COUNT[key]
+
+
+def attention_splits(num_ctas: int, max_context: int, device) -> int:
+    """Into how many CTAs to cut every tile's key range: 1 while the launch fills the GPU by itself, else enough to give
+    every SM a CTA, each with at least two 64-key tiles."""
+    sms = sm_count(device)
     if num_ctas * 2 > sms:
         return 1
     return max(1, min(sms // num_ctas, max_context // 128, 32))
@@ -488,6 +496,23 @@ def paged_attention_kernel(dtype, heads: int, kv_heads: int, dk: int, dv: int, p
     return name, n
 
 
+def paged_attention_flash_forms(dtype, heads: int, kv_heads: int, dk: int, dv: int, page_size: int) -> dict:
+    """The forms of the register-softmax kernel that serve these sizes, each with the most tokens an entry of its ``tiles`` may
+    hold: ``flash`` (64 query rows per CTA: steps with prompt portions) and ``flash_split`` (16 rows whose keys the warps share:
+    single tokens); empty where the general or the older tensor-core kernel has to do (TL_PAGED_FLASH=0 forces that)."""
+    lib = library()
+    if dtype != torch.bfloat16 or any(os.environ.get(v, "1") == "0" for v in ("TL_PAGED_FLASH", "TL_PAGED_MMA")) or not lib.tlb_paged_attention_flash_supported(dk, dv, kv_heads, page_size):
+        return {}
+    sizes = {"flash": int(lib.tlb_paged_attention_flash_tile_tokens(heads, kv_heads, 0)), "flash_split": int(lib.tlb_paged_attention_flash_tile_tokens(heads, kv_heads, 1))}
+    return {name: n for name, n in sizes.items() if n > 0}
+
+
+def flash_splits(num_ctas: int, reach: int, device) -> int:
+    """Into how many CTAs of a cluster to cut every tile's key range: 1 while the launch fills the GPU (two CTAs per SM) by
+    itself, at most 8, each with at least one 64-key tile."""
+    return max(1, min(2 * sm_count(device) // max(num_ctas, 1), -(-reach // 64), 8))
+
+
 def paged_attention_tile_tokens(heads: int, kv_heads: int) -> int:
     """The most tokens an entry of ``tiles`` may hold for the general ``paged_attention`` kernel with these head counts."""
     return paged_attention_kernel(torch.float32, heads, kv_heads, 1, 1, 32)[1]
@@ -554,7 +579,7 @@ def paged_attention(q, slab, block_table, tiles, tok_pos, *, kv_heads: int, dv: 
                     sink: bool = False, gate=None, out=None, kernel: str = "general", max_context: int = 0, head_bias=None, weights: int = 0, keep_first: int = 0):
     """``q [T, H, dk]`` (a view with unit inner stride) against ``slab [P, page, kv_heads * (dk + dv)]`` -> ``out [T, H, dv]``
     (the query's dtype; given, a view with unit inner stride).  ``gate [T, H]`` (a view with unit inner stride): logits of a sigmoid output gate.
-    ``kernel`` and the tile size of ``tiles`` come from ``paged_attention_kernel``.  ``max_context`` (the longest sequence of
+    ``kernel`` and the tile size of ``tiles`` come from ``paged_attention_kernel`` or ``paged_attention_flash_forms``.  ``max_context`` (the longest sequence of
     the step, 0 = unknown) lets the tensor-core kernel split the key range over several CTAs when the launch alone would
     leave SMs idle.  ``head_bias`` (fp32 ``[H]``): with ``sink`` the sink's term is ``exp(head_bias[h])`` instead of ``exp(0)``;
     with ``weights=WEIGHTS_SIGMOID`` there is no softmax, a visible key weighs ``sigmoid(score + head_bias[h])``.  ``keep_first``
@@ -573,6 +598,18 @@ def paged_attention(q, slab, block_table, tiles, tok_pos, *, kv_heads: int, dv: 
         out = torch.empty((T, H, dv), dtype=q.dtype, device=q.device)
     elif out.shape != (T, H, dv) or out.dtype != q.dtype or out.stride(2) != 1:
         raise RuntimeError("paged_attention: out must be [T, H, dv] of the query's dtype with unit inner stride")
+    if kernel in ("flash", "flash_split"):
+        if slab.dtype != torch.bfloat16:
+            raise RuntimeError("paged_attention: the tensor-core kernels take a bfloat16 cache")
+        rows, group = 64 if kernel == "flash" else 16, H // kv_heads
+        reach = min(max_context, int(mask_size) + int(keep_first)) if mask != MASK_CAUSAL else max_context
+        splits = flash_splits(tiles.shape[0] * kv_heads * -(-group // rows), reach, slab.device) if reach else 1
+        _check(library().tlb_paged_attention_flash(_ptr(q), q.stride(0), q.stride(1), _ptr(slab), P, page_size, dk, dv, H, kv_heads, _ptr(block_table),
+                                                   block_table.shape[1], _ptr(tiles), tiles.shape[0], _ptr(tok_pos), int(mask), int(mask_size), int(keep_first),
+                                                   float(scale), float(softcap or 0.0), int(bool(sink)), _ptr(gate), gate.stride(0) if gate is not None else 0,
+                                                   _ptr(out), out.stride(0), out.stride(1), int(kernel == "flash_split"), splits, _ptr(head_bias), int(weights),
+                                                   _stream(q)))
+        return out
     if kernel == "mma":
         if slab.dtype != torch.bfloat16:
             raise RuntimeError("paged_attention: the tensor-core kernel takes a bfloat16 cache")

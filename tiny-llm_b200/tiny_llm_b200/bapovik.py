@@ -119,7 +119,7 @@ class BapovikModel(RaggedDecoderModel):
         max_pages = None if max_tokens is None else -(-int(max_tokens) // page_size)
         self.page_pool = LatentPagedPool(widths, page_size=page_size, dtype=dtype, device=self.device, max_pages=max_pages)
         self.state_pool = StateSlotPool(state_floats, device=self.device, max_slots=max_requests)
-        self.tile_sizes = sorted({layer.attention.tile_tokens for layer in self.layers})
+        self.tile_sizes = sorted({size for layer in self.layers for size in layer.attention.tile_sizes})
 
     @staticmethod
     def _feed_forward(spec, prefix: str, take):

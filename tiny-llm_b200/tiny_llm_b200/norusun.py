@@ -177,7 +177,7 @@ class NorusunModel(RaggedDecoderModel):
         sizes = set()
         for layer in self.layers:
             if layer.attention is not None:
-                sizes.add(layer.attention.tile_tokens)
+                sizes.update(layer.attention.tile_sizes)
             if layer.mixer is not None:
                 sizes.add(blocks.attention_kernel(dtype, layer.mixer.heads, layer.mixer.rank, layer.mixer.rot_dim, page_size)[1])
         self.tile_sizes = sorted(sizes) or [blocks.ATTENTION_TILE_TOKENS]

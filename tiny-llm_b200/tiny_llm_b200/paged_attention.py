@@ -122,8 +122,23 @@ class PagedGroupedAttention:
                 raise ValueError(f"attention: cannot rotate {self.rot['dims']} of {self.dim} entries")
         from extensions_b200.tiny_llm_ext_b200 import blocks
 
-        # the kernel (tensor cores for a bf16 cache of fitting sizes, else the general one) and its work-list granularity
+        # the kernel (tensor cores for a bf16 cache of fitting sizes, else the general one) and its work-list granularity; the
+        # register-softmax kernel's forms, which take over wherever they serve the sizes
         self.kernel, self.tile_tokens = blocks.paged_attention_kernel(self.w_o.dtype, self.heads, self.kv_heads, self.dim, self.vdim, int(page_size))
+        self.forms = blocks.paged_attention_flash_forms(self.w_o.dtype, self.heads, self.kv_heads, self.dim, self.vdim, int(page_size))
+
+    @property
+    def tile_sizes(self) -> list:
+        """The work-list granularities a step's plan has to offer."""
+        return sorted(set(self.forms.values())) if self.forms else [self.tile_tokens]
+
+    def _kernel(self, plan) -> tuple:
+        """(kernel, its work list's granularity) for a step: the form that splits the keys over the warps when every request
+        brings as few rows as one of its tiles holds, the wide one for prompt portions."""
+        if not self.forms:
+            return self.kernel, self.tile_tokens
+        name = "flash_split" if plan.max_tokens <= self.forms.get("flash_split", 0) else "flash"
+        return name, self.forms[name]
 
     @property
     def cache_width(self) -> int:
@@ -158,6 +173,7 @@ class PagedGroupedAttention:
                                   tok_pos=plan.tok_pos, tok_seq=plan.tok_seq, block_table=plan.block_table, slab=slab)
             elif q_norm is not None:
                 blocks.kv_prepare(q3, None, None, q_norm=q_norm, eps=self.eps)
-        return blocks.paged_attention(q3, slab, plan.block_table, plan.tiles_for(self.tile_tokens), plan.tok_pos, kv_heads=G, dv=self.vdim, mask=self.mask,
+        kernel, tile = self._kernel(plan)
+        return blocks.paged_attention(q3, slab, plan.block_table, plan.tiles_for(tile), plan.tok_pos, kv_heads=G, dv=self.vdim, mask=self.mask,
                                       mask_size=self.mask_size, keep_first=self.keep_first, scale=self.scale, softcap=self.softcap, sink=self.sink, gate=gate,
-                                      kernel=self.kernel, max_context=getattr(plan, "max_context", 0), head_bias=self.head_bias, weights=self.weights, out=out)
+                                      kernel=kernel, max_context=getattr(plan, "max_context", 0), head_bias=self.head_bias, weights=self.weights, out=out)

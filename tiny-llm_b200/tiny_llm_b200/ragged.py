@@ -126,6 +126,7 @@ class RaggedPlan:
         self.tiles = self._tiles[sizes[0]]
         self.max_context = max(o.offset for o in owners)  # the longest sequence after this step's append
         self.want_counts = [len(x) for x in wants]
+        self.all_wanted = W == T and all(x == list(range(len(x))) for x in wants)  # the wanted rows are the step's rows, in order
         self.starts = starts
         self.max_tokens = max(len(e.tokens) for e in entries)  # the longest entry of the step
         self.owners = owners

@@ -10,6 +10,7 @@ scheduler use.  A subclass sets ``page_pool`` (a pool with ``slab_version``), ``
 
 from __future__ import annotations
 
+import contextlib
 import os
 
 import torch
@@ -27,7 +28,28 @@ class RaggedDecoderModel:
         # table width); the step's integers are data in one device block.  None = on for CUDA, False = always eager.
         self.use_decode_graph: bool | None = None if os.environ.get(self.graph_env, "1") != "0" else False
         self._graphs: dict = {}
+        self._side, self._forked = None, False  # the second stream of _beside
         self.graph_replays = self.graph_captures = 0
+
+    @contextlib.contextmanager
+    def _beside(self, on: bool = True):
+        """What is queued inside runs on a second stream, after everything queued so far and beside what follows until
+        ``_join``.  It may use tensors made outside; what it makes inside must not be used outside but through memory made
+        outside (an ``out=``), which has to live until the join.  Works under graph capture (a fork and a join)."""
+        if not on or self.device.type != "cuda":
+            yield
+            return
+        if self._side is None:
+            self._side = torch.cuda.Stream(self.device)
+        self._side.wait_stream(torch.cuda.current_stream(self.device))
+        self._forked = True
+        with torch.cuda.stream(self._side):
+            yield
+
+    def _join(self) -> None:
+        if self._forked:
+            torch.cuda.current_stream(self.device).wait_stream(self._side)
+            self._forked = False
 
     def _storage_version(self):
         """Changes whenever device storage that a captured graph addresses has been reallocated."""

@@ -159,7 +159,7 @@ class SenuraxModel(RaggedDecoderModel):
         max_pages = None if max_tokens is None else -(-int(max_tokens) // page_size)
         self.page_pool = LatentPagedPool(widths, page_size=page_size, dtype=dtype, device=self.device, max_pages=max_pages)
         self.state_pool = StateSlotPool(state_floats, device=self.device, max_slots=max_requests)
-        self.tile_sizes = sorted({layer.attention.tile_tokens for layer in self.layers if layer.attention is not None}) or [blocks.ATTENTION_TILE_TOKENS]
+        self.tile_sizes = sorted({size for layer in self.layers if layer.attention is not None for size in layer.attention.tile_sizes}) or [blocks.ATTENTION_TILE_TOKENS]
 
     @staticmethod
     def _rot(spec):

@@ -20,7 +20,7 @@ The model is the framework's usual object (``RaggedDecoderModel``).  A request h
 (``LatentPagedPool``: one slab per layer with keys of its own, rows of ``kv_heads * (dim + vdim)``) and the ids it has run,
 whose newest one the pair embedding of its next portion reads.  Compute dtype bf16 (serving) or fp32 (every product in true
 fp32); embedding sum, residual, norms, scores, softmax and rotation angles are fp32 in both.  A layer's two branches meet in
-one product (``JoinedProjection``), whose fp32 accumulator makes their sum.
+one product (``JoinedProjection``), whose fp32 accumulator makes their sum; small steps run them on two streams.
 """
 
 from __future__ import annotations
@@ -36,6 +36,9 @@ from .mlp import GatedMLP
 from .paged_attention import FusedProjection, JoinedProjection, PagedGroupedAttention
 from .ragged import RaggedPlan
 from .ragged_model import RaggedDecoderModel
+
+
+BESIDE_TOKENS = 128  # steps of up to this many tokens run a layer's two branches side by side: neither fills the GPU
 
 
 class ZalazenLayer:
@@ -102,7 +105,7 @@ class ZalazenModel(RaggedDecoderModel):
         self.head = take("head")
         max_pages = None if max_tokens is None else -(-int(max_tokens) // page_size)
         self.page_pool = LatentPagedPool(widths, page_size=page_size, dtype=dtype, device=self.device, max_pages=max_pages)
-        self.tile_sizes = sorted({layer.attention.tile_tokens for layer in self.layers})
+        self.tile_sizes = sorted({size for layer in self.layers for size in layer.attention.tile_sizes})
 
     @staticmethod
     def _rotation(rot):
@@ -135,10 +138,12 @@ class ZalazenModel(RaggedDecoderModel):
         """What the layer adds to the stream, fp32 ``[T, width]``."""
         T, a = h1.shape[0], layer.attention
         operand, part = layer.out.operand(T)
+        with self._beside(layer.mlp is not None and T <= BESIDE_TOKENS):
+            if layer.mlp is not None:
+                layer.mlp.inner(h2, out=part["down"])
         y = layer.proj(h1)
         a.attend(y["q"], y.get("k"), y.get("v"), y["g"], plan, self.page_pool.slabs[layer.slab_index], out=part["o"].unflatten(1, (a.heads, a.vdim)))
-        if layer.mlp is not None:
-            layer.mlp.inner(h2, out=part["down"])
+        self._join()
         return layer.out(operand)
 
     def _forward_plan(self, plan: RaggedPlan) -> torch.Tensor:
@@ -153,7 +158,7 @@ class ZalazenModel(RaggedDecoderModel):
                 # the layer's sum, fused with the next layer's norms (the model's norm runs on the wanted rows only)
                 following = self.layers[i + 1] if i + 1 < len(self.layers) else None
                 if following is None:
-                    blocks.add_norm(x32, delta, None, None, self.eps)
+                    h1 = blocks.add_norm(x32, delta, None, self.final_norm if plan.all_wanted else None, self.eps)
                 elif following.norm2 is None:
                     h1, h2 = blocks.add_norm(x32, delta, None, following.norm1, self.eps), None
                 else:
@@ -162,8 +167,9 @@ class ZalazenModel(RaggedDecoderModel):
                     self.stream_tap.append(x32.clone())
             if plan.num_want == 0:  # a portion whose logits nobody asked for: the cache is filled, that is all
                 return torch.empty((0, self.vocab_size), dtype=torch.float32, device=self.device)
-            rows = x32.index_select(0, plan.want_rows.long())
-            return linear_wide(blocks.norm_residual(rows, self.final_norm, self.eps), self.head)
+            if not plan.all_wanted:
+                h1 = blocks.norm_residual(x32.index_select(0, plan.want_rows), self.final_norm, self.eps)
+            return linear_wide(h1, self.head)
         finally:
             if exact:
                 torch.backends.cuda.matmul.allow_tf32 = tf32
