@@ -1711,7 +1711,8 @@ def _zalazen_kernels(cfg: dict, device, prompt: int, batch: int, context: int) -
     x, y = torch.randn((rows, D), device=device), torch.randn((rows, D), device=device)
     ms = timed(lambda: blocks.add_norm(x, y, None, w1, eps, w2))
     out["residual_two_norms"] = stream(rows * D * (4 + 4 + 4 + 2 + 2), ms, rows=rows)
-    ms = timed(lambda: blocks.add_norm(x, y, y, w1, eps))
+    z = torch.randn((rows, D), device=device)
+    ms = timed(lambda: blocks.add_norm(x, y, z, w1, eps))
     out["like_add_norm"] = stream(rows * D * (4 + 4 + 4 + 4 + 2), ms, rows=rows)
     few, fy = x[:batch], y[:batch]
     ms = timed(lambda: blocks.add_norm(few, fy, None, w1, eps, w2))
@@ -1747,10 +1748,11 @@ def _zalazen_kernels(cfg: dict, device, prompt: int, batch: int, context: int) -
     del wide, q, k, v, slab
 
     window, keep = cfg["windows"][0]
-    kernel, tile = blocks.paged_attention_kernel(bf, H, G, dk, dv, page)
+    forms = blocks.paged_attention_flash_forms(bf, H, G, dk, dv, page)
+    older = blocks.paged_attention_kernel(bf, H, G, dk, dv, page)
     sink = torch.randn(H, device=device)
 
-    def attention(tokens_per_seq, seqs, ctx, plain=False):
+    def attention(tokens_per_seq, seqs, ctx, kernel, tile, plain=False):
         pages_per = -(-ctx // page)
         slab = torch.randn((seqs * pages_per, page, G * (dk + dv)), dtype=torch.float32, device=device).to(bf)
         table = torch.arange(seqs * pages_per, dtype=torch.int32, device=device).view(seqs, pages_per)
@@ -1764,14 +1766,17 @@ def _zalazen_kernels(cfg: dict, device, prompt: int, batch: int, context: int) -
         return timed(lambda: blocks.paged_attention(q, slab, table, tiles, tok, kv_heads=G, dv=dv, mask=blocks.MASK_WINDOW, mask_size=window, scale=dk ** -0.5,
                                                     gate=gate, out=o, kernel=kernel, max_context=ctx, **more))
 
-    for name, plain in (("window_kept_sink_attention", False), ("like_window_attention", True)):
+    wide, single = ("flash", forms["flash"]), ("flash_split", forms["flash_split"])
+    # the design's attention; the window attention of the closest model, which runs on the same kernel; and the kernel both had before
+    for name, wide_form, single_form, plain in (("window_kept_sink_attention", wide, single, False), ("like_window_attention", wide, single, True),
+                                                ("earlier_kernel_window_kept_sink_attention", older, older, False)):
         kept = 0 if plain else keep
-        ms = attention(prompt, 1, prompt, plain)
+        ms = attention(prompt, 1, prompt, *wide_form, plain)
         seen = sum(min(p + 1, window) + max(0, min(kept, p + 1 - window)) for p in range(prompt))
-        out[name + "_prefill"] = math(2.0 * H * (dk + dv) * seen, ms, kernel=kernel, tokens=prompt, window=window, keep_first=kept)
-        ms = attention(1, batch, context, plain)
+        out[name + "_prefill"] = math(2.0 * H * (dk + dv) * seen, ms, kernel=wide_form[0], tokens=prompt, window=window, keep_first=kept)
+        ms = attention(1, batch, context, *single_form, plain)
         seen = min(context, window) + max(0, min(kept, context - window))
-        out[name + "_decode"] = stream(batch * seen * G * (dk + dv) * 2, ms, kernel=kernel, batch=batch, context=context)
+        out[name + "_decode"] = stream(batch * seen * G * (dk + dv) * 2, ms, kernel=single_form[0], batch=batch, context=context)
     ff = cfg["ff"]
     for n, name in ((rows // 4, "gated_silu"), (batch, "gated_silu_decode")):
         gu, dst = torch.randn((n, 2 * ff), device=device).to(bf), torch.empty((n, H * dv + ff), dtype=bf, device=device)

@@ -15,7 +15,6 @@ from oracle import zalazen as O
 from extensions_b200.tiny_llm_ext_b200 import blocks
 from tiny_llm_b200 import BatchingKvCache, ContinuousBatcher, greedy_generate_ids
 from tiny_llm_b200.models import load_model, model_class
-from tiny_llm_b200.paged_attention import JoinedProjection
 from tiny_llm_b200.positional_encoding import yarn_ramp
 from tiny_llm_b200.ragged import RaggedEntry
 from tiny_llm_b200.synthetic import save_zalazen, synthetic_zalazen, zalazen_config
@@ -137,6 +136,8 @@ def test_rotation_tables_stretched_by_frequency(dev, dims, base, scaling):
 @pytest.mark.parametrize("first,width", [(16, 24), (9, 24), (5, 13), (0, 40)])
 def test_gated_activation_and_attention_meet_in_one_product(dev, dtype, first, width):
     """The activation lands in columns of a wider matrix (neighbours untouched); the joined product equals the sum of both."""
+    from tiny_llm_b200.paged_attention import JoinedProjection
+
     g = torch.Generator().manual_seed(first * 100 + width)
     T, D = 11, 32
     gu = torch.randn(T, 2 * width, generator=g).to(dtype)

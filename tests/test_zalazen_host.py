@@ -11,7 +11,6 @@ import torch
 from oracle import zalazen as O
 from tiny_llm_b200.latent_kv_cache import LatentPagedCache, LatentPagedPool
 from tiny_llm_b200.models import ARCHITECTURES
-from tiny_llm_b200.paged_attention import JoinedProjection
 from tiny_llm_b200.positional_encoding import yarn_ramp
 from tiny_llm_b200.ragged import RaggedEntry, RaggedPlan
 from tiny_llm_b200.state_cache import HybridPagedCache, StateSlotPool
@@ -77,13 +76,39 @@ def test_history_follows_a_rewind_and_a_step_that_was_refused():
     with pytest.raises(RuntimeError, match="exhausted"):
         RaggedPlan([RaggedEntry([1, 2], [a]), RaggedEntry([3] * 8, [b])], "cpu", 4)
     assert list(a.tokens) == [5, 6, 7, 8, 40] and a.offset == 5 and len(b.tokens) == 0
+    with pytest.raises(ValueError, match="wanted place"):           # refused before anything is appended
+        RaggedPlan([RaggedEntry([1, 2], [a], want=[2])], "cpu", 4)
+    with pytest.raises(ValueError, match="once per step"):
+        RaggedPlan([RaggedEntry([1], [a]), RaggedEntry([2], [a])], "cpu", 4)
+    with pytest.raises(ValueError, match="at least one token"):
+        RaggedPlan([RaggedEntry([1], [a]), RaggedEntry([], [b])], "cpu", 4)
+    assert list(a.tokens) == [5, 6, 7, 8, 40] and a.offset == 5 and b.offset == 0
     a.append_slots(2)                                             # filled by something that is no step: no ids known
     assert RaggedPlan([RaggedEntry([50], [a])], "cpu", 4).seq_prev.tolist() == [-1]
     assert list(a.tokens) == [5, 6, 7, 8, 40, -1, -1, 50]
 
 
+def test_plan_rows_of_unequal_entries():
+    pool = LatentPagedPool([8], page_size=4, device="cpu", dtype=torch.float32)
+    a, b, c = (LatentPagedCache(pool) for _ in range(3))
+    RaggedPlan([RaggedEntry([9] * 6, [b])], "cpu", 4)
+    plan = RaggedPlan([RaggedEntry([1, 2, 3, 4, 5], [a], want=[4, 0]), RaggedEntry([6], [b], want=[]), RaggedEntry([7, 8], [c])], "cpu", [2, 4])
+    assert plan.ids.tolist() == [1, 2, 3, 4, 5, 6, 7, 8] and plan.tok_pos.tolist() == [0, 1, 2, 3, 4, 6, 0, 1] and plan.tok_seq.tolist() == [0] * 5 + [1, 2, 2]
+    assert plan.want_rows.tolist() == [4, 0, 7] and plan.want_counts == [2, 0, 1] and not plan.all_wanted and plan.max_tokens == 5 and plan.max_context == 7
+    assert plan.tiles_for(2).tolist() == [[0, 2, 0], [2, 2, 0], [4, 1, 0], [5, 1, 1], [6, 2, 2]]
+    assert plan.tiles_for(4).tolist() == [[0, 4, 0], [4, 1, 0], [5, 1, 1], [6, 2, 2]]
+    assert plan.seq_info.tolist() == [[0, 5, 0, -1], [5, 1, 6, -1], [6, 2, 0, -1]] and plan.seq_prev.tolist() == [-1, 9, -1]
+    assert plan.block_table.tolist() == [a.page_ids, b.page_ids, c.page_ids + [-1]]
+    plan = RaggedPlan([RaggedEntry([1], [c]), RaggedEntry([3], [a], want=[0, 0]), RaggedEntry([2], [b], want=[])], "cpu", [2, 4])
+    assert plan.tok_pos.tolist() == [2, 5, 7] and plan.want_rows.tolist() == [0, 1, 1] and plan.tiles_for(4).tolist() == [[0, 1, 0], [1, 1, 1], [2, 1, 2]]
+    assert not plan.all_wanted and RaggedPlan([RaggedEntry([1, 2], [a], want=range(2)), RaggedEntry([1], [b])], "cpu", 4).all_wanted
+    assert not RaggedPlan([RaggedEntry([1, 2], [a], want=[1, 0])], "cpu", 4).all_wanted
+
+
 # ---------------------------------------------------------------------------------------------- small product parts
 def test_joined_projection_keeps_one_copy_and_sums_its_parts():
+    from tiny_llm_b200.paged_attention import JoinedProjection
+
     g = torch.Generator().manual_seed(1)
     w1, w2 = torch.randn(6, 10, generator=g), torch.randn(6, 7, generator=g)
     j = JoinedProjection([("a", w1), ("b", w2)])

@@ -27,6 +27,7 @@ constexpr int kFWarps = 4;
 constexpr int kFKeys = 64;   // keys per tile
 constexpr int kFSplits = 8;  // most CTAs of a cluster
 constexpr float kLog2e = 1.4426950408889634f;
+constexpr uint32_t kOnes = 0x3F803F80u;  // two bf16 ones
 
 struct FlashArgs {
     const bf16 *q;
@@ -44,15 +45,14 @@ struct FlashArgs {
     bf16 *out;
     long long o_token, o_head;
     const float *head_bias;
-    int weights, k_stride, v_stride, q_wide /* 16-byte query loads */, o_pairs /* 4-byte output stores */;
+    int weights, k_stride, q_wide /* 16-byte query loads */, o_pairs /* 4-byte output stores */;
 };
 
-__device__ __forceinline__ void f_ldm_x4(uint32_t (&r)[4], const void *p) {
-    uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
+__device__ __forceinline__ uint32_t f_addr(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void f_ldm_x4(uint32_t (&r)[4], uint32_t a) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
 }
-__device__ __forceinline__ void f_ldm_x4_trans(uint32_t (&r)[4], const void *p) {
-    uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
+__device__ __forceinline__ void f_ldm_x4_trans(uint32_t (&r)[4], uint32_t a) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
 }
 __device__ __forceinline__ void f_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
@@ -60,8 +60,7 @@ __device__ __forceinline__ void f_mma(float (&c)[4], const uint32_t (&a)[4], uin
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-__device__ __forceinline__ void f_cp16(void *dst, const void *src) {
-    uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
+__device__ __forceinline__ void f_cp16(uint32_t d, const void *src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
 }
 __device__ __forceinline__ float f_ex2(float x) {
@@ -78,17 +77,20 @@ __device__ __forceinline__ float f_tanh(float x) {
 // 2^(a - b) where b is a running maximum: 0 for a = -infinity, also when both are
 __device__ __forceinline__ float f_weight(float a, float b) { return a == -INFINITY ? 0.f : f_ex2(a - b); }
 
-// NV: units of 16 value columns; SPLIT: the form (see above).
-template <int NV, bool SPLIT>
-__global__ void __launch_bounds__(kFWarps * 32)
+// NV: units of 16 value columns; SPLIT: the form (see above); KT: units of 16 query / key columns when known (the queries then
+// stay in registers), 0 = any number.
+template <int NV, bool SPLIT, int KT>
+__global__ void __launch_bounds__(kFWarps * 32, NV <= 8 ? 2 : 1)
 paged_attention_flash_kernel(const FlashArgs A) {
     constexpr int ROWS = SPLIT ? 16 : 16 * kFWarps;
     constexpr int NT = SPLIT ? 2 : kFKeys / 8;  // 8-key score tiles per warp
     constexpr int COLS = NV * 16;
+    constexpr int VS = COLS + 8;                       // value row stride; (stride / 8) odd: conflict-free ldmatrix rows
+    const int KS = KT ? KT * 16 + 8 : A.k_stride;      // query / key row stride
     extern __shared__ __align__(16) unsigned char smem_raw[];
-    bf16 *sq = reinterpret_cast<bf16 *>(smem_raw);  // [ROWS][k_stride]
-    bf16 *skv = sq + ROWS * A.k_stride;             // [2] x ([64][k_stride] keys | [64][v_stride] values)
-    const int buf_elems = kFKeys * (A.k_stride + A.v_stride);
+    bf16 *sq = reinterpret_cast<bf16 *>(smem_raw);     // [ROWS][KS]; with KT only until the queries are in registers
+    bf16 *skv = KT ? sq : sq + ROWS * KS;              // [2] x ([64][KS] keys | [64][VS] values)
+    const int buf_elems = kFKeys * (KS + VS);
 
     const int group = A.heads / A.kv_heads, hp = A.hp, parts = (group + hp - 1) / hp;
     const int g = blockIdx.y / parts, part = blockIdx.y % parts;
@@ -99,19 +101,19 @@ paged_attention_flash_kernel(const FlashArgs A) {
     const int k_pieces = A.dk / 8, per_row = k_pieces + A.dv / 8;  // 16-byte pieces of a key row, of a cache row's share of this head
 
     // padding must read as zero in every product: query rows without a token, columns of Q and K past dk
-    for (int i = threadIdx.x; i < (ROWS * A.k_stride + 2 * buf_elems) / 8; i += blockDim.x) reinterpret_cast<uint4 *>(sq)[i] = make_uint4(0, 0, 0, 0);
+    for (int i = threadIdx.x; i < ((KT ? 0 : ROWS * KS) + 2 * buf_elems) / 8; i += blockDim.x) reinterpret_cast<uint4 *>(sq)[i] = make_uint4(0, 0, 0, 0);
     __syncthreads();
     if (A.q_wide) {
         for (int i = threadIdx.x; i < ROWS * k_pieces; i += blockDim.x) {
             const int r = i / k_pieces, piece = i - r * k_pieces, tq = r / hp, hh = r - tq * hp;
             if (tq < count && hh < nheads)
-                *reinterpret_cast<uint4 *>(sq + r * A.k_stride + piece * 8) =
+                *reinterpret_cast<uint4 *>(sq + r * KS + piece * 8) =
                     *reinterpret_cast<const uint4 *>(A.q + (size_t)(first + tq) * A.q_token + (size_t)(head0 + hh) * A.q_head + piece * 8);
         }
     } else {
         for (int i = threadIdx.x; i < ROWS * A.dk; i += blockDim.x) {
             const int r = i / A.dk, d = i - r * A.dk, tq = r / hp, hh = r - tq * hp;
-            if (tq < count && hh < nheads) sq[r * A.k_stride + d] = A.q[(size_t)(first + tq) * A.q_token + (size_t)(head0 + hh) * A.q_head + d];
+            if (tq < count && hh < nheads) sq[r * KS + d] = A.q[(size_t)(first + tq) * A.q_token + (size_t)(head0 + hh) * A.q_head + d];
         }
     }
 
@@ -129,39 +131,47 @@ paged_attention_flash_kernel(const FlashArgs A) {
 
     const int32_t *table = A.block_table + (size_t)seq * A.max_pages;
     const size_t row_width = (size_t)A.kv_heads * (A.dk + A.dv), k_off = (size_t)g * A.dk, v_off = (size_t)A.kv_heads * A.dk + (size_t)g * A.dv;
-    const int step_rows = (int)blockDim.x / per_row, step_pieces = (int)blockDim.x % per_row;
+    // a warp copies whole rows: `span` lanes a row (a power of two), 32 / span rows at a time, a lane the same 16-byte pieces of
+    // every row it takes
+    int span = 32;
+    while (span / 2 >= per_row) span /= 2;
+    const int my_row = warp * (32 / span) + lane / span, my_piece = lane % span, rows_at_once = kFWarps * (32 / span);
     auto stage = [&](int tile, int buf) {
-        bf16 *sk = skv + buf * buf_elems, *sv = sk + kFKeys * A.k_stride;
+        const uint32_t sk = f_addr(skv + buf * buf_elems), sv = sk + kFKeys * KS * 2;
         const int k0 = tile_key(tile);
-        const bf16 *src[2];  // a page holds a multiple of 32 keys: each half of a tile lies in one page
-        int valid[2];
 #pragma unroll
-        for (int h = 0; h < 2; ++h) {
+        for (int h = 0; h < 2; ++h) {  // a page holds a multiple of 32 keys: each half of a tile lies in one page
             const int key = k0 + 32 * h;
             const int page = key <= hi ? table[key / A.page_size] : -1;
             const bool ok = page >= 0 && page < A.num_pages;  // a bad table entry reads as zeros
-            src[h] = A.slab + ((size_t)(ok ? page : 0) * A.page_size + key % A.page_size) * row_width;
-            valid[h] = ok ? min(32, hi - key + 1) : 0;
-        }
-        int j = (int)threadIdx.x / per_row, piece = (int)threadIdx.x % per_row;
-        while (j < kFKeys) {
-            const bool is_v = piece >= k_pieces;
-            const int col = (is_v ? piece - k_pieces : piece) * 8, h = j >> 5, jj = j & 31;
-            bf16 *dst = is_v ? sv + j * A.v_stride + col : sk + j * A.k_stride + col;
-            if (jj < (h ? valid[1] : valid[0])) f_cp16(dst, (h ? src[1] : src[0]) + (size_t)jj * row_width + (is_v ? v_off : k_off) + col);
-            else *reinterpret_cast<uint4 *>(dst) = make_uint4(0, 0, 0, 0);
-            j += step_rows, piece += step_pieces;
-            if (piece >= per_row) piece -= per_row, ++j;
+            const int valid = ok ? min(32, hi - key + 1) : 0;
+            for (int piece = my_piece; piece < per_row; piece += 32) {
+                const bool is_v = piece >= k_pieces;
+                const int col = (is_v ? piece - k_pieces : piece) * 8, stride = is_v ? VS : KS;
+                const bf16 *src = A.slab + ((size_t)(ok ? page : 0) * A.page_size + key % A.page_size + my_row) * row_width + (is_v ? v_off : k_off) + col;
+                uint32_t dst = (is_v ? sv : sk) + ((32 * h + my_row) * stride + col) * 2;
+                const size_t src_step = (size_t)rows_at_once * row_width;
+                const uint32_t dst_step = rows_at_once * stride * 2;
+                for (int j = my_row; j < 32; j += rows_at_once, src += src_step, dst += dst_step) {
+                    if (j < valid) f_cp16(dst, src);
+                    else asm volatile("st.shared.v4.b32 [%0], {%1, %1, %1, %1};" ::"r"(dst), "r"(0) : "memory");
+                }
+            }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
 
-    // the two rows of this thread's quad: what they may see ([see_lo, see_hi] and keys below keep_first), their running maximum
-    // (in powers of two) and this thread's share of the running sum
+    // scores enter the exponential as 2^(s * mult - maximum * mult): s as the product leaves it where the maximum may be taken
+    // over that (a softmax without a cap, a positive scale), else s already scaled and capped and mult = 1
+    const float scale2 = A.scale * kLog2e, cap_in = A.softcap > 0.f ? A.scale / A.softcap : 0.f, cap_out = A.softcap * kLog2e;
+    const bool raw = A.softcap <= 0.f && A.scale > 0.f && A.weights == 0;
+    const float mult = raw ? scale2 : 1.f;
+    // the two rows of this thread's quad: what they may see ([see_lo, see_hi] and keys below keep_first) and their running
+    // maximum; the running sums are one more accumulator tile, P times a matrix of ones
     const int row0 = SPLIT ? 0 : warp * 16;
     const bool opens = blockIdx.z == 0 && (!SPLIT || warp == 0);  // who counts the sink (or the sigmoid form's constant sum), once
     int see_lo[2], see_hi[2];
-    float m[2], l[2], hb[2];
+    float m[2], hb[2];
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
         const int r = row0 + gq + 8 * h, tq = r / hp, hh = r - tq * hp;
@@ -170,8 +180,7 @@ paged_attention_flash_kernel(const FlashArgs A) {
         see_hi[h] = live ? p : -1;
         see_lo[h] = !live ? 0x7fffffff : A.mask == 1 ? max(0, p - A.mask_size + 1) : A.mask == 2 ? p / A.mask_size * A.mask_size : 0;
         hb[h] = A.head_bias && live ? A.head_bias[head0 + hh] * kLog2e : 0.f;
-        m[h] = A.weights == 1 ? 0.f : A.sink && opens ? hb[h] : -INFINITY;
-        l[h] = opens && t4 == 0 && (A.sink || A.weights == 1) ? 1.f : 0.f;
+        m[h] = A.weights == 1 ? 0.f : A.sink && opens ? hb[h] / mult : -INFINITY;
     }
     const int first_kept = A.mask == 1 ? A.keep_first : 0;
     // over the warp's live rows: tokens ascend with the row, so the first row's range starts first and the last one's ends last
@@ -187,41 +196,58 @@ paged_attention_flash_kernel(const FlashArgs A) {
         }
         warp_lo = a, warp_hi = b, all_lo = c, all_hi = d;
     }
-    const float scale2 = A.scale * kLog2e, cap_in = A.softcap > 0.f ? A.scale / A.softcap : 0.f, cap_out = A.softcap * kLog2e;
 
-    float acc[2 * NV][4];
+    float acc[2 * NV][4], sums[4];
+    sums[0] = sums[1] = sums[2] = sums[3] = opens && (A.sink || A.weights == 1) ? 1.f : 0.f;
 #pragma unroll
     for (int i = 0; i < 2 * NV; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
 
-    const int ksteps = (A.dk + 15) / 16;
+    const int ksteps = KT ? KT : (A.dk + 15) / 16;
     __syncthreads();  // the zero fill and the queries are in place before the first copies land
+    const uint32_t q_at = f_addr(sq + (row0 + (lane & 15)) * KS + (lane >> 4) * 8);
+    uint32_t qf[KT ? KT : 1][4];
+    if constexpr (KT > 0) {
+#pragma unroll
+        for (int ks = 0; ks < KT; ++ks) f_ldm_x4(qf[ks], q_at + ks * 32);
+        __syncthreads();
+        for (int i = threadIdx.x; i < ROWS * KS / 8; i += blockDim.x) reinterpret_cast<uint4 *>(sq)[i] = make_uint4(0, 0, 0, 0);  // key padding again
+        __syncthreads();
+    }
+    const uint32_t k_at = ((SPLIT ? warp * 16 : 0) + (lane & 7) + (lane >> 4) * 8) * KS * 2 + ((lane >> 3) & 1) * 16;
+    const uint32_t v_at = kFKeys * KS * 2 + ((SPLIT ? warp * 16 : 0) + (lane & 7) + ((lane >> 3) & 1) * 8) * VS * 2 + (lane >> 4) * 16;
     if (tile_begin < tile_end) stage(tile_begin, 0);
     for (int tile = tile_begin; tile < tile_end; ++tile) {
         const int buf = (tile - tile_begin) & 1;
-        const bf16 *sk = skv + buf * buf_elems, *sv = sk + kFKeys * A.k_stride;
+        const uint32_t base_at = f_addr(skv + buf * buf_elems);
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();  // this tile has landed, and every warp is done with the previous one: its buffer may be refilled
         if (tile + 1 < tile_end) stage(tile + 1, buf ^ 1);
         const int key0 = tile_key(tile) + (SPLIT ? warp * 16 : 0), key_end = key0 + NT * 8 - 1;
         if (key0 > warp_hi || (key_end < warp_lo && key0 >= first_kept)) continue;  // no row of the warp sees any of its keys
-        const int kr = SPLIT ? warp * 16 : 0;
 
         float s[NT][4];
 #pragma unroll
         for (int i = 0; i < NT; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
         {
-            const bf16 *qa = sq + (row0 + (lane & 15)) * A.k_stride + (lane >> 4) * 8;
-            const bf16 *kb = sk + (kr + (lane & 7) + (lane >> 4) * 8) * A.k_stride + ((lane >> 3) & 1) * 8;
-#pragma unroll 2
-            for (int ks = 0; ks < ksteps; ++ks) {
-                uint32_t a[4];
-                f_ldm_x4(a, qa + ks * 16);
+            const uint32_t kb = base_at + k_at;
+            auto step = [&](int ks, const uint32_t (&a)[4]) {
 #pragma unroll
                 for (int n = 0; n < NT / 2; ++n) {
                     uint32_t b[4];
-                    f_ldm_x4(b, kb + n * 16 * A.k_stride + ks * 16);
+                    f_ldm_x4(b, kb + n * 32 * KS + ks * 32);
                     f_mma(s[2 * n], a, b[0], b[1]);
                     f_mma(s[2 * n + 1], a, b[2], b[3]);
+                }
+            };
+            if constexpr (KT > 0) {
+#pragma unroll
+                for (int ks = 0; ks < KT; ++ks) step(ks, qf[ks]);
+            } else {
+#pragma unroll 2
+                for (int ks = 0; ks < ksteps; ++ks) {
+                    uint32_t a[4];
+                    f_ldm_x4(a, q_at + ks * 32);
+                    step(ks, a);
                 }
             }
         }
@@ -230,7 +256,7 @@ paged_attention_flash_kernel(const FlashArgs A) {
             for (int i = 0; i < NT; ++i)
 #pragma unroll
                 for (int e = 0; e < 4; ++e) s[i][e] = cap_out * f_tanh(s[i][e] * cap_in);
-        } else {
+        } else if (!raw) {
 #pragma unroll
             for (int i = 0; i < NT; ++i)
 #pragma unroll
@@ -258,20 +284,15 @@ paged_attention_flash_kernel(const FlashArgs A) {
                 for (int i = 0; i < NT; ++i) mx = fmaxf(mx, fmaxf(s[i][2 * h], s[i][2 * h + 1]));
                 mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
                 mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-                const float alpha = f_weight(m[h], mx), base = mx == -INFINITY ? 0.f : mx;
+                const float base = mx == -INFINITY ? 0.f : __fmul_rn(mx, mult);
+                const float alpha = m[h] == -INFINITY ? 0.f : f_ex2(__fmul_rn(m[h], mult) - base);  // exactly 1 where the maximum stays
                 m[h] = mx;
-                float sum = 0.f;
 #pragma unroll
-                for (int i = 0; i < NT; ++i)
-#pragma unroll
-                    for (int e = 2 * h; e < 2 * h + 2; ++e) {
-                        s[i][e] = __bfloat162float(__float2bfloat16_rn(f_ex2(s[i][e] - base)));  // numerator and denominator see the same rounded weights
-                        sum += s[i][e];
-                    }
-                l[h] = l[h] * alpha + sum;
+                for (int i = 0; i < NT; ++i) s[i][2 * h] = f_ex2(fmaf(s[i][2 * h], mult, -base)), s[i][2 * h + 1] = f_ex2(fmaf(s[i][2 * h + 1], mult, -base));
                 if (__any_sync(0xffffffffu, alpha != 1.f)) {
 #pragma unroll
                     for (int i = 0; i < 2 * NV; ++i) acc[i][2 * h] *= alpha, acc[i][2 * h + 1] *= alpha;
+                    sums[2 * h] *= alpha, sums[2 * h + 1] *= alpha;
                 }
             }
         }
@@ -279,20 +300,16 @@ paged_attention_flash_kernel(const FlashArgs A) {
         for (int kk = 0; kk < NT / 2; ++kk) {
             const uint32_t a[4] = {tl::pack2<bf16>(s[2 * kk][0], s[2 * kk][1]), tl::pack2<bf16>(s[2 * kk][2], s[2 * kk][3]),
                                    tl::pack2<bf16>(s[2 * kk + 1][0], s[2 * kk + 1][1]), tl::pack2<bf16>(s[2 * kk + 1][2], s[2 * kk + 1][3])};
-            const bf16 *vb = sv + (kr + kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * A.v_stride + (lane >> 4) * 8;
+            if (A.weights == 0) f_mma(sums, a, kOnes, kOnes);  // numerator and denominator see the same rounded weights
+            const uint32_t vb = base_at + v_at + kk * 32 * VS;
 #pragma unroll
             for (int n = 0; n < NV; ++n) {
                 uint32_t b[4];
-                f_ldm_x4_trans(b, vb + n * 16);
+                f_ldm_x4_trans(b, vb + n * 32);
                 f_mma(acc[2 * n], a, b[0], b[1]);
                 f_mma(acc[2 * n + 1], a, b[2], b[3]);
             }
         }
-    }
-#pragma unroll
-    for (int h = 0; h < 2; ++h) {
-        l[h] += __shfl_xor_sync(0xffffffffu, l[h], 1);
-        l[h] += __shfl_xor_sync(0xffffffffu, l[h], 2);
     }
     auto factor = [&](int r, float sum) {  // what a row's sums are multiplied by on their way out
         const int tq = r / hp, hh = r - tq * hp;
@@ -313,7 +330,7 @@ paged_attention_flash_kernel(const FlashArgs A) {
         for (int h = 0; h < 2; ++h) {
             const int r = row0 + gq + 8 * h;
             if (!row_live(r)) continue;
-            const float inv = factor(r, l[h]);
+            const float inv = factor(r, sums[2 * h]);
 #pragma unroll
             for (int i = 0; i < 2 * NV; ++i) {
                 const int col = i * 8 + 2 * t4;
@@ -336,7 +353,7 @@ paged_attention_flash_kernel(const FlashArgs A) {
 #pragma unroll
             for (int i = 0; i < 2 * NV; ++i)
                 *reinterpret_cast<float2 *>(so + ((size_t)p * ROWS + r) * COLS + i * 8 + 2 * t4) = make_float2(acc[i][2 * h], acc[i][2 * h + 1]);
-            if (t4 == 0) sm[p * ROWS + r] = m[h], sl[p * ROWS + r] = l[h];
+            if (t4 == 0) sm[p * ROWS + r] = m[h] == -INFINITY ? m[h] : m[h] * mult, sl[p * ROWS + r] = sums[2 * h];
         }
     }
     cg::cluster_group cluster = cg::this_cluster();
@@ -372,11 +389,11 @@ static int f_units(int dv) {
     return u <= 2 ? 2 : u <= 4 ? 4 : u <= 6 ? 6 : u <= 8 ? 8 : u <= 12 ? 12 : 16;
 }
 
-template <int NV, bool SPLIT>
+template <int NV, bool SPLIT, int KT>
 static int f_launch(const FlashArgs &args, int num_tiles, int splits, cudaStream_t st) {
-    auto kernel = paged_attention_flash_kernel<NV, SPLIT>;
+    auto kernel = paged_attention_flash_kernel<NV, SPLIT, KT>;
     const int rows = SPLIT ? 16 : 16 * kFWarps;
-    const size_t smem = (size_t)(rows * args.k_stride + 2 * kFKeys * (args.k_stride + args.v_stride)) * sizeof(bf16);
+    const size_t smem = (size_t)((KT ? 0 : rows * args.k_stride) + 2 * kFKeys * (args.k_stride + NV * 16 + 8)) * sizeof(bf16);
     if (smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return tl::fail(TL_ECUDA, "paged_attention_flash: %s", cudaGetErrorString(e));
@@ -440,19 +457,19 @@ int tlb_paged_attention_flash(const void *q, long long q_token, long long q_head
     a.mask = mask, a.mask_size = mask_size, a.keep_first = keep_first, a.scale = scale, a.softcap = softcap, a.sink = sink;
     a.gate = (const bf16 *)gate, a.g_token = g_token, a.out = (bf16 *)out, a.o_token = o_token, a.o_head = o_head, a.head_bias = head_bias, a.weights = weights;
     a.k_stride = ceil_div(dk, 16) * 16 + 8;  // (stride / 8) odd: conflict-free ldmatrix rows
-    a.v_stride = nv * 16 + 8;
     a.q_wide = tl::aligned16(q) && q_token % 8 == 0 && q_head % 8 == 0;
     a.o_pairs = (uintptr_t)out % 4 == 0 && o_token % 2 == 0 && o_head % 2 == 0;
     cudaStream_t st = as_stream(stream);
     int rc = TL_OK;
-#define TLB_FLASH(N) rc = split_keys ? f_launch<N, true>(a, num_tiles, splits, st) : f_launch<N, false>(a, num_tiles, splits, st)
+#define TLB_FLASH(N, K) rc = split_keys ? f_launch<N, true, K>(a, num_tiles, splits, st) : f_launch<N, false, K>(a, num_tiles, splits, st)
+    const int kt = ceil_div(dk, 16);
     switch (nv) {
-        case 2: TLB_FLASH(2); break;
-        case 4: TLB_FLASH(4); break;
-        case 6: TLB_FLASH(6); break;
-        case 8: TLB_FLASH(8); break;
-        case 12: TLB_FLASH(12); break;
-        default: TLB_FLASH(16); break;
+        case 2: TLB_FLASH(2, 0); break;
+        case 4: if (kt == 4) TLB_FLASH(4, 4); else TLB_FLASH(4, 0); break;
+        case 6: TLB_FLASH(6, 0); break;
+        case 8: if (kt == 8) TLB_FLASH(8, 8); else TLB_FLASH(8, 0); break;
+        case 12: TLB_FLASH(12, 0); break;
+        default: TLB_FLASH(16, 0); break;
     }
 #undef TLB_FLASH
     if (rc != TL_OK) return rc;

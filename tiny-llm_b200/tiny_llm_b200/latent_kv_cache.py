@@ -13,6 +13,7 @@ from __future__ import annotations
 
 from array import array
 
+import numpy as np
 import torch
 
 from .kv_cache import TinyKvCache
@@ -96,13 +97,13 @@ class LatentPagedCache(TinyKvPagedCache):
         super().__init__(pool)
         self.tokens = array("q")
 
-    def record_tokens(self, ids) -> None:
-        """The ids of the newest ``len(ids)`` slots, after ``append_slots``."""
+    def record_tokens(self, ids: np.ndarray) -> None:
+        """The ids (int64) of the newest ``len(ids)`` slots, after ``append_slots``."""
         at = self.offset - len(ids)
         if at > len(self.tokens):  # slots filled by something that is no step: their ids are unknown
             self.tokens.extend([-1] * (at - len(self.tokens)))
         del self.tokens[at:]
-        self.tokens.extend(int(t) for t in ids)
+        self.tokens.frombytes(ids.tobytes())
 
     def rewind(self, n: int):
         super().rewind(n)

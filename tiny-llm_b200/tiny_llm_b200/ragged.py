@@ -42,35 +42,37 @@ class RaggedPlan:
         """``max_pages`` fixes the block table's width (at least what the longest request needs) and ``into`` names a
         preallocated int32 device block to upload into: a captured graph reads the same addresses every step."""
         sizes = sorted({int(tile)} if isinstance(tile, int) else {int(t) for t in tile})
-        owners = []
-        for e in entries:
-            if len(e.tokens) == 0:
-                raise ValueError("a ragged entry needs at least one token")
-            owner = getattr(e.cache[0], "owner", e.cache[0])
-            if any(owner is o for o in owners):
-                raise ValueError("a request may appear once per step")
-            owners.append(owner)
+        owners = [getattr(e.cache[0], "owner", e.cache[0]) for e in entries]
+        counts = [len(e.tokens) for e in entries]
+        if min(counts) == 0:
+            raise ValueError("a ragged entry needs at least one token")
+        if len({id(o) for o in owners}) < len(owners):
+            raise ValueError("a request may appear once per step")
+        wants = [[n - 1] if e.want is None else list(e.want) for e, n in zip(entries, counts)]
+        for n, places in zip(counts, wants):  # checked before anything is appended
+            for place in places:
+                if not 0 <= place < n:
+                    raise ValueError(f"wanted place {place} is outside the entry's {n} tokens")
+        tokens = [np.asarray(e.tokens, dtype=np.int64) for e in entries]
         starts = [o.offset for o in owners]
         done = []
         try:
-            for o, e in zip(owners, entries):
-                o.append_slots(len(e.tokens))
-                done.append((o, len(e.tokens)))
+            for o, n in zip(owners, counts):
+                o.append_slots(n)
+                done.append((o, n))
         except Exception:
             for o, n in done:  # all-or-nothing: give the pages of this step back
                 o.rewind(n)
             raise
-        T = sum(len(e.tokens) for e in entries)
-        S = len(entries)
+        T, S = sum(counts), len(entries)
         needed = max(o.num_pages for o in owners)
         if max_pages is not None and max_pages < needed:
             for o, n in done:
                 o.rewind(n)
             raise ValueError(f"block table of {max_pages} pages, {needed} needed")
         max_pages = needed if max_pages is None else max_pages
-        wants = [list(e.want) if e.want is not None else [len(e.tokens) - 1] for e in entries]
         W = sum(len(w) for w in wants)
-        n_tiles = {size: sum(-(-len(e.tokens) // size) for e in entries) for size in sizes}
+        n_tiles = {size: sum(-(-n // size) for n in counts) for size in sizes}
         total = self.block_ints(T, W, S, max_pages, sum(n_tiles.values()))
         host = torch.empty(max(total, 1), dtype=torch.int32, pin_memory=torch.cuda.is_available() and torch.device(device).type == "cuda")
         buf = host.numpy()
@@ -84,28 +86,34 @@ class RaggedPlan:
             at += 3 * n_tiles[size]
         info = buf[at : at + 4 * S].reshape(S, 4)
         prev = buf[at + 4 * S : at + 5 * S]
-        tile_rows = {size: [] for size in sizes}
-        t = w = 0
-        for s, (e, o, start) in enumerate(zip(entries, owners, starts)):
-            n = len(e.tokens)
-            ids[t : t + n] = np.asarray(e.tokens, dtype=np.int64)
-            pos[t : t + n] = np.arange(start, start + n, dtype=np.int64)
-            seq[t : t + n] = s
-            for place in wants[s]:
-                if not 0 <= place < n:
-                    raise ValueError(f"wanted place {place} is outside the entry's {n} tokens")
-                want[w] = t + place
-                w += 1
-            for size in sizes:
-                tile_rows[size] += [(t + first, min(size, n - first), s) for first in range(0, n, size)]
+        work = [(size, buf[start : start + 3 * n].reshape(n, 3)) for size, (start, n) in tile_at.items()]
+        row_of = np.arange(S)
+        firsts = np.cumsum([0] + counts[:-1])
+        ids[:] = np.concatenate(tokens) if S > 1 else tokens[0]
+        seq[:] = np.repeat(row_of, counts) if T > S else row_of
+        info[:, 0], info[:, 1], info[:, 2] = firsts, counts, starts
+        info[:, 3] = [getattr(o, "state_slot", -1) for o in owners]
+        histories = [getattr(o, "tokens", None) for o in owners]
+        prev[:] = [h[start - 1] if h is not None and 0 < start <= len(h) else -1 for h, start in zip(histories, starts)]
+        for s, o in enumerate(owners):
             table[s, : o.num_pages] = o.page_ids
-            info[s] = (t, n, start, getattr(o, "state_slot", -1))
-            history = getattr(o, "tokens", None)
-            prev[s] = history[start - 1] if history is not None and 0 < start <= len(history) else -1
-            t += n
-        for size in sizes:
-            start, n = tile_at[size]
-            buf[start : start + 3 * n] = np.asarray(tile_rows[size], dtype=np.int32).reshape(-1)
+        if T == S:  # one token per sequence
+            pos[:] = starts
+            want[:] = [s for s, places in enumerate(wants) for _ in places]
+            for _, rows in work:
+                rows[:, 0], rows[:, 1], rows[:, 2] = row_of, 1, row_of
+        else:
+            at_row, w = {size: 0 for size in sizes}, 0
+            for s, (t, n, start) in enumerate(zip(firsts.tolist(), counts, starts)):
+                pos[t : t + n] = np.arange(start, start + n)
+                if wants[s]:
+                    want[w : w + len(wants[s])] = np.asarray(wants[s]) + t
+                    w += len(wants[s])
+                for size, rows in work:
+                    offsets = np.arange(0, n, size)
+                    part = rows[at_row[size] : at_row[size] + len(offsets)]
+                    part[:, 0], part[:, 1], part[:, 2] = t + offsets, np.minimum(size, n - offsets), s
+                    at_row[size] += len(offsets)
         self.num_tokens, self.num_seqs, self.num_want, self.max_pages = T, S, W, max_pages
         self.h2d_bytes = total * 4
         if into is None:
@@ -128,11 +136,11 @@ class RaggedPlan:
         self.want_counts = [len(x) for x in wants]
         self.all_wanted = W == T and all(x == list(range(len(x))) for x in wants)  # the wanted rows are the step's rows, in order
         self.starts = starts
-        self.max_tokens = max(len(e.tokens) for e in entries)  # the longest entry of the step
+        self.max_tokens = max(counts)  # the longest entry of the step
         self.owners = owners
-        for o, e in zip(owners, entries):  # from here on the step runs: what it consumes cannot be taken back from a recurrent state
+        for o, ran in zip(owners, tokens):  # from here on the step runs: what it consumes cannot be taken back from a recurrent state
             if hasattr(o, "record_tokens"):
-                o.record_tokens(e.tokens)
+                o.record_tokens(ran)
             if hasattr(o, "ran_offset"):
                 o.ran_offset = o.offset
 
