@@ -111,7 +111,8 @@ def test_a_cluster_shares_the_key_range(dev, kernel, kind, size, sink):
                 close(got, want[lo : lo + n], 2e-2)
     finally:
         blocks.flash_splits = original
-    assert blocks.flash_splits(1, 700, dev) == 8 and blocks.flash_splits(1, 65, dev) == 2 and blocks.flash_splits(10**6, 10**6, dev) == 1
+    assert blocks.flash_splits(1, 700, None, dev) == 8 and blocks.flash_splits(1, 700, 65, dev) == 2 and blocks.flash_splits(10**6, 10**6, None, dev) == 1
+    assert {blocks.flash_splits(1, n, None, dev) for n in (1, 5, 128, 256)} == {4}   # the same over a captured step's range of contexts
 
 
 @pytest.mark.parametrize("kernel", ["flash", "flash_split"])

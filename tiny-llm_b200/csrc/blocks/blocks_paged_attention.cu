@@ -329,7 +329,8 @@ __device__ __forceinline__ void qk_unpack8(uint4 u, float (&x)[8]) {
 }
 
 template <bool INTERLEAVED>
-__global__ void qk_whole_prepare_wide_kernel(bf16 *q, long long q_token, int heads, const bf16 *__restrict__ q_norm, const bf16 *__restrict__ k,
+__global__ void __launch_bounds__(1024)
+qk_whole_prepare_wide_kernel(bf16 *q, long long q_token, int heads, const bf16 *__restrict__ q_norm, const bf16 *__restrict__ k,
                                              long long k_token, const bf16 *__restrict__ v, long long v_token, int kv_heads, int dk, int dv,
                                              const bf16 *__restrict__ k_norm, float eps, int rot_dims, const int32_t *__restrict__ tok_pos,
                                              const int32_t *__restrict__ tok_seq, const int32_t *__restrict__ block_table, int max_pages, int num_pages,
@@ -337,44 +338,29 @@ __global__ void qk_whole_prepare_wide_kernel(bf16 *q, long long q_token, int hea
     __shared__ float partial[2][32];
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int q_chunks = heads * dk / 8, k_chunks = k ? kv_heads * dk / 8 : 0, v_chunks = k ? kv_heads * dv / 8 : 0;
-    bf16 *dst = nullptr;
-    if (k != nullptr) {
-        const int pos = tok_pos[t];
-        const int page = block_table[(size_t)tok_seq[t] * max_pages + pos / page_size];
-        if (page >= 0 && page < num_pages) dst = slab + ((size_t)page * page_size + pos % page_size) * ((size_t)kv_heads * (dk + dv));
-    }
     int c = threadIdx.x;
     const bool is_q = c < q_chunks, is_k = !is_q && c < q_chunks + k_chunks, is_v = !is_q && !is_k && c < q_chunks + k_chunks + v_chunks;
     if (is_k) c -= q_chunks;
     if (is_v) c -= q_chunks + k_chunks;
-    float x[8], y[8], g[8], gy[8], cs[8], sn[8];
-    bool turned = false, low = false;
-    if (is_v) {
-        if (dst) *reinterpret_cast<uint4 *>(dst + (size_t)kv_heads * dk + c * 8) = *reinterpret_cast<const uint4 *>(v + (size_t)t * v_token + c * 8);
-    }
+    const bf16 *src = is_q ? q + (size_t)t * q_token : is_k ? k + (size_t)t * k_token : v + (size_t)t * v_token, *w = is_q ? q_norm : k_norm;
+    const int e = c * 8 % dk, half = rot_dims / 2;  // the chunk's place in its head
+    const bool turned = (is_q || is_k) && e < rot_dims, low = e < half;
+    const int other = c * 8 + (INTERLEAVED ? 0 : low ? half : -half);  // the columns its own are rotated with
+    // before the row's sum is known only raw columns are held (few registers: many rows in flight), the rest is read afterwards
+    uint4 raw = make_uint4(0, 0, 0, 0), partner = raw;
+    if (is_q || is_k || is_v) raw = *reinterpret_cast<const uint4 *>(src + c * 8);
+    if (!INTERLEAVED && turned) partner = *reinterpret_cast<const uint4 *>(src + other);
+    float x[8], g[8];
+    qk_unpack8(raw, x);
     float sq = 0.f;
-    const bf16 *src = is_q ? q + (size_t)t * q_token : k + (is_k ? (size_t)t * k_token : 0), *w = is_q ? q_norm : k_norm;
-    if (is_q || is_k) {
-        const int e = c * 8 % dk, half = rot_dims / 2;  // the chunk's place in its head
-        qk_unpack8(*reinterpret_cast<const uint4 *>(src + c * 8), x);
-        if (w) qk_unpack8(*reinterpret_cast<const uint4 *>(w + c * 8), g);
-        turned = e < rot_dims;
-        if (turned) {
-            const int i0 = INTERLEAVED ? e / 2 : (e < half ? e : e - half);
-            low = e < half;
-            const float4 *cp = reinterpret_cast<const float4 *>(rope_cos + (size_t)t * half + i0), *sp = reinterpret_cast<const float4 *>(rope_sin + (size_t)t * half + i0);
-            const float4 c0 = cp[0], s0 = sp[0];
-            cs[0] = c0.x, cs[1] = c0.y, cs[2] = c0.z, cs[3] = c0.w, sn[0] = s0.x, sn[1] = s0.y, sn[2] = s0.z, sn[3] = s0.w;
-            if (!INTERLEAVED) {
-                const float4 c1 = cp[1], s1 = sp[1];
-                cs[4] = c1.x, cs[5] = c1.y, cs[6] = c1.z, cs[7] = c1.w, sn[4] = s1.x, sn[5] = s1.y, sn[6] = s1.z, sn[7] = s1.w;
-                const int other = c * 8 + (low ? half : -half);
-                qk_unpack8(*reinterpret_cast<const uint4 *>(src + other), y);
-                if (w) qk_unpack8(*reinterpret_cast<const uint4 *>(w + other), gy);
-            }
-        }
 #pragma unroll
-        for (int j = 0; j < 8; ++j) sq = fmaf(x[j], x[j], sq);
+    for (int j = 0; j < 8; ++j) sq = fmaf(x[j], x[j], sq);
+    bf16 *dst = nullptr;  // the token's cache row: a chain of loads that runs beside the row's own
+    if (is_k || is_v) {
+        const int pos = tok_pos[t];
+        const int page = block_table[(size_t)tok_seq[t] * max_pages + pos / page_size];
+        if (page >= 0 && page < num_pages) dst = slab + ((size_t)page * page_size + pos % page_size) * ((size_t)kv_heads * (dk + dv));
+        if (is_v && dst) *reinterpret_cast<uint4 *>(dst + (size_t)kv_heads * dk + c * 8) = raw;
     }
     const float a = warp_sum(is_q ? sq : 0.f), b = warp_sum(is_k ? sq : 0.f);
     if (lane == 0) partial[0][warp] = a, partial[1][warp] = b;
@@ -383,20 +369,38 @@ __global__ void qk_whole_prepare_wide_kernel(bf16 *q, long long q_token, int hea
     float total = 0.f;
     for (int i = 0; i < (int)(blockDim.x >> 5); ++i) total += partial[is_q ? 0 : 1][i];
     const float inv = w ? 1.0f / sqrtf(total / (float)((is_q ? heads : kv_heads) * dk) + eps) : 1.f;
+    auto normed = [&](float (&z)[8], int col) {
+        if (w == nullptr) return;
+        qk_unpack8(*reinterpret_cast<const uint4 *>(w + col), g);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) x[j] = x[j] * inv * (w ? g[j] : 1.f);
+        for (int j = 0; j < 8; ++j) z[j] = z[j] * inv * g[j];
+    };
+    qk_unpack8(raw, x);
+    normed(x, c * 8);
     if (turned) {
+        const int i0 = INTERLEAVED ? e / 2 : (low ? e : e - half);
+        const float4 *cp = reinterpret_cast<const float4 *>(rope_cos + (size_t)t * half + i0), *sp = reinterpret_cast<const float4 *>(rope_sin + (size_t)t * half + i0);
         if (INTERLEAVED) {
+            const float4 c0 = cp[0], s0 = sp[0];
+            const float cs[4] = {c0.x, c0.y, c0.z, c0.w}, sn[4] = {s0.x, s0.y, s0.z, s0.w};
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const float u = x[2 * j], z = x[2 * j + 1];
                 x[2 * j] = u * cs[j] - z * sn[j], x[2 * j + 1] = z * cs[j] + u * sn[j];
             }
         } else {
+            float y[8];
+            qk_unpack8(partner, y);
+            normed(y, other);
 #pragma unroll
-            for (int j = 0; j < 8; ++j) {
-                const float z = y[j] * inv * (w ? gy[j] : 1.f);
-                x[j] = low ? x[j] * cs[j] - z * sn[j] : x[j] * cs[j] + z * sn[j];
+            for (int q4 = 0; q4 < 2; ++q4) {
+                const float4 c4 = cp[q4], s4 = sp[q4];
+                const float cs[4] = {c4.x, c4.y, c4.z, c4.w}, sn[4] = {s4.x, s4.y, s4.z, s4.w};
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const float z = y[4 * q4 + j], u = x[4 * q4 + j];
+                    x[4 * q4 + j] = low ? u * cs[j] - z * sn[j] : u * cs[j] + z * sn[j];
+                }
             }
         }
     }

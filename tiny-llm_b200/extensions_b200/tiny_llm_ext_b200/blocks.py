@@ -507,9 +507,12 @@ def paged_attention_flash_forms(dtype, heads: int, kv_heads: int, dk: int, dv: i
     return {name: n for name, n in sizes.items() if n > 0}
 
 
-def flash_splits(num_ctas: int, reach: int, device) -> int:
+def flash_splits(num_ctas: int, max_context: int, most, device) -> int:
     """Into how many CTAs of a cluster to cut every tile's key range: 1 while the launch fills the GPU (two CTAs per SM) by
-    itself, at most 8, each with at least one 64-key tile."""
+    itself, at most 8, with a 64-key tile for each by the longest context rounded up to a power of two (from 256) and the most
+    keys a mask lets through (``most``, None = all).  Rounded up, so that a captured step and an eager one cut alike."""
+    reach = max(256, 1 << (max(max_context, 1) - 1).bit_length())
+    reach = reach if most is None else min(reach, int(most))
     return max(1, min(2 * sm_count(device) // max(num_ctas, 1), -(-reach // 64), 8))
 
 
@@ -602,8 +605,8 @@ def paged_attention(q, slab, block_table, tiles, tok_pos, *, kv_heads: int, dv: 
         if slab.dtype != torch.bfloat16:
             raise RuntimeError("paged_attention: the tensor-core kernels take a bfloat16 cache")
         rows, group = 64 if kernel == "flash" else 16, H // kv_heads
-        reach = min(max_context, int(mask_size) + int(keep_first)) if mask != MASK_CAUSAL else max_context
-        splits = flash_splits(tiles.shape[0] * kv_heads * -(-group // rows), reach, slab.device) if reach else 1
+        most = int(mask_size) + int(keep_first) if mask != MASK_CAUSAL else None
+        splits = flash_splits(tiles.shape[0] * kv_heads * -(-group // rows), max_context, most, slab.device) if max_context else 1
         _check(library().tlb_paged_attention_flash(_ptr(q), q.stride(0), q.stride(1), _ptr(slab), P, page_size, dk, dv, H, kv_heads, _ptr(block_table),
                                                    block_table.shape[1], _ptr(tiles), tiles.shape[0], _ptr(tok_pos), int(mask), int(mask_size), int(keep_first),
                                                    float(scale), float(softcap or 0.0), int(bool(sink)), _ptr(gate), gate.stride(0) if gate is not None else 0,
