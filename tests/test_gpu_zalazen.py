@@ -545,6 +545,25 @@ def test_random_stacks_and_sizes_in_random_schedules(dev, seed):
     assert not model.page_pool.used_page_ids
 
 
+@pytest.mark.parametrize("seed", range(8))
+def test_random_stacks_in_the_serving_dtype(dev, seed):
+    """Sizes that take the register-softmax kernel's forms and sizes that do not, in bfloat16: whole, and decoded after a prompt."""
+    g = torch.Generator().manual_seed(2000 + seed)
+    pick = lambda *options: options[int(torch.randint(0, len(options), (1,), generator=g))]
+    kv_heads, dim = pick(1, 2, 3), pick(8, 24, 32, 64, 128, 144)
+    config = zalazen_config(pattern=pick("AdSd", "AnAdSd", "AdAd"), width=pick(56, 96, 128), vocab=pick(64, 101), heads=kv_heads * pick(1, 3, 4, 20), kv_heads=kv_heads,
+                            dim=dim, vdim=pick(8, 12, 32, 64, 104, 128, 200), windows=tuple((pick(3, 31, 64, 65, 128), pick(0, 1, 32, 65)) for _ in range(3)),
+                            rot_dims=pick(2, dim // 8 * 8, dim // 4 * 2), ff=pick(24, 64, 75), buckets=pick(0, 64, 1009))
+    tensors = synthetic_zalazen(config, seed=seed)
+    model = model_class("Zalazen").from_checkpoint(config, tensors, dtype=torch.bfloat16, device=dev, max_tokens=6 * 64)
+    prompt = ids_for(200, config["vocab"], seed)
+    want = O.forward(prompt, tensors, config)
+    whole = run_schedule(model, {"a": prompt}, [[("a", 200)]])["a"]
+    assert rows_match(whole, want, torch.bfloat16), config
+    got = run_schedule(model, {"a": prompt}, [[("a", 97)], [("a", 2)], [("a", 65)]] + [[("a", 1)]] * 36)["a"]
+    assert rows_match(got, want, torch.bfloat16), config
+
+
 def test_long_decoding(dev):
     """500 single-token steps after a two-token prompt (graph replays over growing block tables, windows sliding along), against
     the plain model."""
