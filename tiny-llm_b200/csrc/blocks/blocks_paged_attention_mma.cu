@@ -1,5 +1,6 @@
 // Grouped-query attention over the paged cache on the tensor cores (bf16 cache, mma.sync m16n8k16, fp32 accumulation and
-// softmax): the bf16 serving path of blocks_paged_attention.cu, same arguments and masks.
+// softmax): same arguments and masks as blocks_paged_attention.cu.  blocks_paged_attention_flash.cu takes its place in the
+// models' steps unless it is switched off (TL_PAGED_FLASH=0).
 //
 // A CTA takes 32 query rows = a run of consecutive tokens of one sequence x the query heads of ONE key/value head (up to
 // 32 of them) and streams every 32-key tile of that head through shared memory once for all of them: keys into one
