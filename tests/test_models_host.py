@@ -200,3 +200,35 @@ def test_dispatch_model_and_operator_dispatch_rules(tiny, cpu_ext, monkeypatch):
     assert seen == [(8, True, False), (9, True, True)]
     with pytest.raises(ValueError, match="at most 8 input rows"):
         quantized_matvec_custom(w.scales, w.biases, 128, 4, torch.zeros(9, 128, dtype=torch.bfloat16), w.weight, True)
+
+
+def test_nothing_is_collected_while_a_graph_is_captured(monkeypatch):
+    """Collecting a dropped model that holds graphs would invalidate a capture under way: the collector waits, and is as it was
+    afterwards, also when the captured step raises."""
+    import contextlib
+    import gc
+
+    from tiny_llm_b200 import graphs
+
+    seen = []
+
+    @contextlib.contextmanager
+    def fake(graph, **kwargs):
+        seen.append((graph, kwargs))
+        yield
+
+    monkeypatch.setattr(graphs.torch.cuda, "graph", fake)
+    with graphs.capture("g", stream="s"):
+        assert not gc.isenabled()
+    assert gc.isenabled() and seen == [("g", {"stream": "s"})]
+    with pytest.raises(ValueError):
+        with graphs.capture("g"):
+            raise ValueError
+    assert gc.isenabled()
+    gc.disable()
+    try:
+        with graphs.capture("g"):
+            pass
+        assert not gc.isenabled()
+    finally:
+        gc.enable()

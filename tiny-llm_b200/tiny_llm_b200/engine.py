@@ -34,6 +34,7 @@ import torch
 
 from extensions_b200 import tiny_llm_ext_b200 as ext
 
+from .graphs import capture
 from .kv_cache import BatchingKvCache
 from .paged_kv_cache import TinyKvPagedCache
 
@@ -317,11 +318,11 @@ class DecodeEngine:
                 forward()
             self._stream.synchronize()
             self._graph = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(self._graph, stream=self._stream):
+            with capture(self._graph, stream=self._stream):
                 forward()
             self._graph_loop = torch.cuda.CUDAGraph()
             launched = ext.launch_count()
-            with torch.cuda.graph(self._graph_loop, stream=self._stream, pool=self._graph.pool()):
+            with capture(self._graph_loop, stream=self._stream, pool=self._graph.pool()):
                 forward()
                 ext.decode_advance(self.tokens, self.next_tokens, self.offsets, self.context_lens, self.out_log, self.step_counter)
             # kernels of libtiny_llm_b200.so recorded into one self-advancing step
@@ -334,7 +335,7 @@ class DecodeEngine:
                     forward(rows)
                 self._stream.synchronize()
                 g = torch.cuda.CUDAGraph()
-                with torch.cuda.graph(g, stream=self._stream, pool=self._graph.pool()):
+                with capture(g, stream=self._stream, pool=self._graph.pool()):
                     forward(rows)
                 self._graphs[rows] = g
         torch.cuda.current_stream(self.device).wait_stream(self._stream)
@@ -682,7 +683,7 @@ class PrefillEngine:
             self._stream.synchronize()
             self._graph = torch.cuda.CUDAGraph()
             launched = ext.launch_count()
-            with torch.cuda.graph(self._graph, stream=self._stream):
+            with capture(self._graph, stream=self._stream):
                 self._forward()
             self.kernels_per_chunk = ext.launch_count() - launched
         torch.cuda.current_stream(self.device).wait_stream(self._stream)

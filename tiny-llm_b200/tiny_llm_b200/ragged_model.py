@@ -15,6 +15,7 @@ import os
 
 import torch
 
+from .graphs import capture
 from .kv_cache import BatchingKvCache
 from .ragged import RaggedEntry, RaggedPlan
 
@@ -100,7 +101,7 @@ class RaggedDecoderModel:
             drop_workspaces = getattr(torch._C, "_cuda_clearCublasWorkspaces", lambda: None)
             drop_workspaces()
             try:
-                with torch.cuda.graph(graph):
+                with capture(graph):
                     state["logits"] = self._forward_plan(plan)
             finally:
                 drop_workspaces()
