@@ -120,13 +120,14 @@ size_t tlb_latent_attention_mma_workspace(int num_tiles, int heads, int rank, in
  * q [T, heads, dk] and out [T, heads, dv] are views with token / head strides in elements.  Token t sees key j <= tok_pos[t]
  * and, mask 1: tok_pos[t] - j < mask_size (sliding window) or j < keep_first (kept first positions; 0 = none); mask 2: j / mask_size == tok_pos[t] / mask_size (chunks counted
  * from position 0); mask 0: all.  score = scale * q.k, then softcap * tanh(score / softcap) when softcap > 0; sink != 0 adds
- * exp(0) to the softmax's denominator; gate != NULL multiplies head h's output by sigmoid(gate[t * g_token + h]).
+ * exp(0) to the softmax's denominator; gate != NULL multiplies head h's output by sigmoid(gate[t * g_token + h]), or, gate_wide,
+ * entry d of it by sigmoid(gate[t * g_token + h * dv + d]).
  * tiles [num_tiles, 3] as for latent attention, cut to at most tlb_paged_attention_tile_tokens(heads, kv_heads) tokens. */
 int tlb_paged_attention_tile_tokens(int heads, int kv_heads);
 int tlb_paged_attention(const void *q, long long q_token, long long q_head, const void *slab, int num_pages, int page_size, int dk, int dv,
                         int heads, int kv_heads, const int32_t *block_table, int max_pages, const int32_t *tiles, int num_tiles,
                         const int32_t *tok_pos, int mask, int mask_size, int keep_first, float scale, float softcap, int sink, const void *gate,
-                        long long g_token, void *out, long long o_token, long long o_head, const float *head_bias, int weights, int dtype,
+                        long long g_token, int gate_wide, void *out, long long o_token, long long o_head, const float *head_bias, int weights, int dtype,
                         void *stream);
 /* head_bias [heads] fp32 (or NULL): with sink != 0 the sink's term is exp(head_bias[h]) instead of exp(0).  weights 1: no
  * softmax, a visible key weighs sigmoid(score + head_bias[h]) and nothing is normalised over the keys (no sink, no cap). */
@@ -138,7 +139,7 @@ int tlb_paged_attention_mma_supported(int dk, int dv, int kv_heads, int page_siz
 int tlb_paged_attention_mma(const void *q, long long q_token, long long q_head, const void *slab, int num_pages, int page_size, int dk, int dv,
                             int heads, int kv_heads, const int32_t *block_table, int max_pages, const int32_t *tiles, int num_tiles,
                             const int32_t *tok_pos, int mask, int mask_size, int keep_first, float scale, float softcap, int sink, const void *gate,
-                            long long g_token, void *out, long long o_token, long long o_head, int splits, void *workspace,
+                            long long g_token, int gate_wide, void *out, long long o_token, long long o_head, int splits, void *workspace,
                             size_t workspace_bytes, const float *head_bias, int weights, void *stream);
 /* splits > 1 cuts every tile's key range over that many CTAs (few query rows, long key ranges) and a second launch merges the
  * partial sums; workspace: tlb_paged_attention_mma_workspace(...) bytes, no initialisation needed. */
@@ -151,8 +152,8 @@ int tlb_paged_attention_flash_tile_tokens(int heads, int kv_heads, int split_key
 int tlb_paged_attention_flash_supported(int dk, int dv, int kv_heads, int page_size);
 int tlb_paged_attention_flash(const void *q, long long q_token, long long q_head, const void *slab, int num_pages, int page_size, int dk, int dv, int heads,
                               int kv_heads, const int32_t *block_table, int max_pages, const int32_t *tiles, int num_tiles, const int32_t *tok_pos,
-                              int mask, int mask_size, int keep_first, float scale, float softcap, int sink, const void *gate, long long g_token, void *out,
-                              long long o_token, long long o_head, int split_keys, int splits, const float *head_bias, int weights, void *stream);
+                              int mask, int mask_size, int keep_first, float scale, float softcap, int sink, const void *gate, long long g_token, int gate_wide,
+                              void *out, long long o_token, long long o_head, int split_keys, int splits, const float *head_bias, int weights, void *stream);
 /* Before that attention: per-head RMS norm (plain weight [dk]) of the queries in place (q_norm != NULL) and of the keys
  * (k_norm != NULL), and the token's keys and values stored at its slot of the cache (k != NULL). */
 int tlb_kv_prepare(void *q, long long q_token, long long q_head, int heads, const void *q_norm, const void *k, long long k_token, long long k_head,
@@ -190,19 +191,30 @@ int tlb_decay_scan(const void *q, long long q_token, long long q_head, const voi
                    const float *rope_cos, const float *rope_sin, int rope_dims, int rope_interleaved, float q_scale, int heads,
                    int dk, int dv, const int32_t *seq_info, int num_seqs, int max_tokens_per_seq, float *state, long long slot_stride,
                    int num_slots, float *out, void *workspace, size_t workspace_bytes, int decay_kind, const void *a_log, const void *bonus,
-                   int qk_heads, const void *skip, int dtype, void *stream);
+                   int qk_heads, const void *skip, int v_cols, int dtype, void *stream);
 /* decay_kind 0: as above.  2: alpha = exp(-exp(z + z_bias)) per key channel.  3: one decay per head and token,
  * alpha = exp(-exp(a_log[h]) dt), dt = softplus(z[t, h] + z_bias[h]) (z [T, heads]), and the token's key is multiplied by dt
- * (a discretised state-space step; a_log [heads] in `dtype`).  qk_heads (0 = heads): q and k have that many heads, head h
+ * (a discretised state-space step; a_log [heads] in `dtype`).  4: z [T, heads, 2] gives one (decay, key factor) pair per head
+ * and token.  v_cols (0 = dv): v has that many columns per head; in the state's columns from there on v reads as 1, so column
+ * v_cols of the output is the decayed sum of the keys times q (a normaliser).  qk_heads (0 = heads): q and k have that many heads, head h
  * reads h / (heads / qk_heads).  skip [heads] (`dtype`, or NULL): out += skip[h] v.  bonus [heads, dk] (`dtype`, or NULL): the
  * read-out comes before the update and weighs the token's own k v^T by it, out = (S + diag(bonus) k v^T)^T q, then S is
  * updated. */
 /* out[t, h, :] = o[t, h, :] / rms(o[t, h, :]) * w * act(gate[t, h, :]) (w NULL = no weight; gate rows g_token apart, NULL = no
  * gate; act 0 = the gate as it is, 1 = silu, 2 = sigmoid); o fp32 [tokens, heads, dv], out `dtype` [tokens, heads * dv].
  * wide_weight: w is [heads * dv], each head its own part, instead of [dv]; gate_first: the gate multiplies o BEFORE the
- * norm, out = n / rms(n) * w with n = o * act(gate). */
+ * norm, out = n / rms(n) * w with n = o * act(gate).  o_row (0 = dv): entries between two rows of o.  floor [tokens, heads] (NULL =
+ * none): o is first divided by max(|o[t, h, dv]|, floor[t, h]) + den_eps, the entry behind a row's dv being a normaliser. */
 int tlb_head_norm_gate(const float *o, const void *w, float eps, const void *gate, long long g_token, int act, void *out, int tokens, int heads,
-                       int dv, int wide_weight, int gate_first, int dtype, void *stream);
+                       int dv, int wide_weight, int gate_first, int o_row, const float *floor, float den_eps, int dtype, void *stream);
+/* The scalar part of a gated matrix memory (mLSTM), per sequence and head along its tokens, m = 0 at position 0:
+ *   i = cap tanh((zi + bias[h]) / cap), f = log_sigmoid(cap tanh((zf + bias[heads + h]) / cap)), m' = max(f + m, i)
+ *   step[t, h] = (exp(f + m - m'), exp(i - m')), floor[t, h] = exp(-m')
+ * (zi | zf) = z [T, 2 * heads] fp32 rows z_token apart, or, z == NULL, the products of hin [T, dim] (rows h_token apart) with
+ * w [2 * heads, dim], made by the kernel (for steps of one or two tokens a sequence).  state: the slot's [heads] block of m. */
+int tlb_matrix_memory_gates(const float *z, long long z_token, const void *hin, long long h_token, const void *w, int dim, const void *bias, float cap,
+                            int heads, const int32_t *seq_info, int num_seqs, int max_tokens_per_seq, float *state, long long slot_stride, int num_slots,
+                            float *step, float *floor, int dtype, void *stream);
 
 /* Gated delta rule, state in fp32 slots.  Per sequence and head S [dk, dv], token by token:
  *   S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  out = S^T q
@@ -256,9 +268,11 @@ int tlb_shift_mix(const void *h, long long h_token, const void *mu, int parts, i
 /* Router: logits = W h + b in fp32 (h, W, b stored in `dtype`; b may be NULL), the `top` largest per token (lower index
  * wins a tie).  scoring 0: weights = softmax over the chosen logits; 1: weights = sigmoid of each chosen logit, not
  * renormalised; 2: scores = softmax over ALL logits, the choice is made by score + choice_bias (`dtype` [experts] or NULL),
- * weights = the chosen scores / (their sum + 1e-20) * weight_scale.  idx [tokens, top] int32, gate [tokens, top] fp32. */
+ * weights = the chosen scores / (their sum + 1e-20) * weight_scale.  group_count > 0: the outputs form that many equal runs of
+ * neighbours, and only those of the group_keep runs with the largest best choice score may be chosen.  aux_w [dim] (NULL =
+ * none): aux[t] = sigmoid(aux_w . h[t]), fp32, beside the routing.  idx [tokens, top] int32, gate [tokens, top] fp32. */
 int tlb_moe_route(const void *h, const void *w, const void *b, int tokens, int dim, int experts, int top, int scoring, const void *choice_bias,
-                  float weight_scale, int32_t *idx, float *gate, int dtype, void *stream);
+                  float weight_scale, int group_count, int group_keep, const void *aux_w, float *aux, int32_t *idx, float *gate, int dtype, void *stream);
 
 /* Rows per expert tile of the grouped products: 32, or 64 for the tensor-core kernels (bf16, reduction length % 8 == 0)
  * when experts get many rows (half the weight traffic per row). */
@@ -269,10 +283,11 @@ long long tlb_moe_max_rows(int tokens, int top, int experts, int tile_rows);
  * counters [2] = {tiles in use, rows in use}.  One launch, no host involvement. */
 int tlb_moe_sort(const int32_t *idx, int tokens, int top, int experts, int tile_rows, int32_t *sorted_pair, int32_t *tile_expert,
                  int32_t *counters, void *stream);
-/* inter[row, :] = act(Wg[e] h[token(row)]) * (Wu[e] h[token(row)]); Wg, Wu [experts, ff, dim]; inter [max_rows, ff]. */
+/* inter[row, :] = act(Wg[e] h[token(row)]) * (Wu[e] h[token(row)]); Wg, Wu [experts, ff, dim]; inter [max_rows, ff]; act, limit and
+ * slope as for tlb_gated_act. */
 int tlb_moe_gate_up(const void *h, const void *wg, const void *wu, const int32_t *sorted_pair, const int32_t *tile_expert,
-                    const int32_t *counters, int tokens, int top, int experts, int tile_rows, int dim, int ff, int act, void *inter,
-                    int dtype, void *stream);
+                    const int32_t *counters, int tokens, int top, int experts, int tile_rows, int dim, int ff, int act, float limit,
+                    float slope, void *inter, int dtype, void *stream);
 /* Experts without a gate: inter[row, :] = act(Wu[e] a[src(row)]) with a = h (token rows, rows_are_pairs = 0) or one row per
  * (token, choice) pair (rows_are_pairs = 1).  act 0 = silu, 1 = gelu (tanh form), 2 = squared relu. */
 int tlb_moe_up(const void *a, const void *wu, const int32_t *sorted_pair, const int32_t *tile_expert, const int32_t *counters, int tokens,
@@ -282,12 +297,26 @@ int tlb_moe_scale_rows(const void *h, const float *gate, void *out, int tokens, 
 /* pair_out[pair, :] = Wd[e] inter[row, :] (fp32); Wd [experts, dim, ff]. */
 int tlb_moe_down(const void *inter, const void *wd, const int32_t *sorted_pair, const int32_t *tile_expert, const int32_t *counters,
                  int tokens, int top, int experts, int tile_rows, int dim, int ff, float *pair_out, int dtype, void *stream);
-/* y[t,:] = sum_k gate[t,k] * pair_out[t*top+k,:] (+ shared[t,:] if shared != NULL, stored in `dtype`), fp32, in choice order;
+/* y[t,:] = sum_k gate[t,k] * pair_out[t*top+k,:] (+ shared_gate[t] * shared[t,:] if shared != NULL, stored in `dtype`; shared_gate
+ * NULL: 1), fp32, in choice order;
  * gate == NULL: every weight is 1.  idx != NULL: a choice with idx[t,k] >= experts is an identity expert (the router has
  * more outputs than there are experts): its output is the token's input h[t,:] (`dtype`), and the grouped products, given
  * `experts` as their count, skip it. */
-int tlb_moe_combine(const float *pair_out, const float *gate, const void *shared, const int32_t *idx, int experts, const void *h, float *y,
+int tlb_moe_combine(const float *pair_out, const float *gate, const void *shared, const float *shared_gate, const int32_t *idx, int experts, const void *h, float *y,
                     int tokens, int top, int dim, int dtype, void *stream);
+
+/* Elementwise bounded norms n(x) = w tanh(alpha x) + b (w, b `dtype` [dim]) around the sublayers of an fp32 stream x [rows, dim];
+ * "next" gives h = n_next(x) rounded to `dtype` (h NULL: none), "post" what a sublayer's output passes on its way into x.
+ * embed: x = n_post(table[ids]).  step: x += n_post(y + y_bias) (y fp32, y_bias `dtype` or NULL).  rows: h = n(x[row_ids[r]])
+ * (row_ids NULL: r), x unchanged.  moe_combine_tanh: x += n_post(y), y the sum of tlb_moe_combine (h_in: the experts' input). */
+int tlb_tanh_embed(const int32_t *ids, const void *table, int vocab, float *x, float post_alpha, const void *post_w, const void *post_b,
+                   float next_alpha, const void *next_w, const void *next_b, void *h, int rows, int dim, int dtype, void *stream);
+int tlb_tanh_step(float *x, const float *y, const void *y_bias, float post_alpha, const void *post_w, const void *post_b, float next_alpha,
+                  const void *next_w, const void *next_b, void *h, int rows, int dim, int dtype, void *stream);
+int tlb_tanh_rows(const float *x, const int32_t *row_ids, float alpha, const void *w, const void *b, void *h, int rows, int dim, int dtype, void *stream);
+int tlb_moe_combine_tanh(float *x, const float *pair_out, const float *gate, const void *shared, const float *shared_gate, const int32_t *idx, int experts,
+                         const void *h_in, int top, float post_alpha, const void *post_w, const void *post_b, float next_alpha, const void *next_w,
+                         const void *next_b, void *h, int rows, int dim, int dtype, void *stream);
 
 /* Row-wise arg-max of fp32 logits [rows, vocab] (lowest index wins a tie). */
 int tlb_argmax_rows(const float *logits, int32_t *out, int rows, int vocab, void *stream);

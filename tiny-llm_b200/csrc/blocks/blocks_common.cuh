@@ -40,6 +40,37 @@ __device__ __forceinline__ void rope_angle(int pos, int i, int dims, double log2
     s = (float)sn;
 }
 
+__device__ __forceinline__ float sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
+__device__ __forceinline__ float log_sigmoid(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
+
+__device__ __forceinline__ float act_apply(float z, int act) {
+    if (act == 0) return z / (1.0f + expf(-z));
+    float inner = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+    return 0.5f * z * (1.0f + tanhf(inner));
+}
+
+// The inside of a gated feed-forward: act(g) * u, or (act 3) the clamped form, the gate bounded from above and the other half on
+// both sides: g sigmoid(slope g) (u + 1).
+__device__ __forceinline__ float gated_pair(float g, float u, int act, float limit, float slope) {
+    if (act == 3) {
+        g = fminf(g, limit), u = fminf(fmaxf(u, -limit), limit);
+        return g / (1.0f + expf(-slope * g)) * (u + 1.0f);
+    }
+    return act_apply(g, act) * u;
+}
+
+// 4 consecutive elements of a row as floats (one 8- or 16-byte access)
+__device__ __forceinline__ float4 load4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
+__device__ __forceinline__ float4 load4(const bf16 *p) {
+    uint2 u = *reinterpret_cast<const uint2 *>(p);
+    float2 a = tl::unpack2<bf16>(u.x), b = tl::unpack2<bf16>(u.y);
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void store4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
+__device__ __forceinline__ void store4(bf16 *p, float4 v) {
+    *reinterpret_cast<uint2 *>(p) = make_uint2(tl::pack2<bf16>(v.x, v.y), tl::pack2<bf16>(v.z, v.w));
+}
+
 }  // namespace tlb
 
 #define TLB_DISPATCH(dtype, name, ...)                                               \

@@ -24,8 +24,6 @@ constexpr int kLaCols = 32;    // state columns per CTA
 constexpr int kLaLanes = 4;    // lanes per column
 constexpr int kLaSegment = TLB_DECAY_SCAN_SEGMENT;  // positions per segment of a long portion
 
-__device__ __forceinline__ float log_sigmoid(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
-
 // Segment c of a sequence's new tokens [p0, p0 + n): cut at the multiples of kLaSegment in ABSOLUTE positions, so that
 // where a prompt was cut into steps does not move the cuts.  Returns false when the sequence has no segment c.
 __device__ __forceinline__ bool la_segment(int p0, int n, int c, int &lo, int &hi, int &nseg) {
@@ -47,7 +45,9 @@ __device__ __forceinline__ bool la_segment(int p0, int n, int c, int &lo, int &h
 //
 // decay_kind chooses where the decay comes from: 0 = sigmoid(z + bias)^(1/tau) per key channel, or head_decay; 2 = exp(-exp(z + bias))
 // per key channel; 3 = one number per head and token, exp(-exp(a_log[h]) dt) with dt = softplus(z[t, h] + bias[h]), and the
-// token's key is multiplied by dt (a discretised state-space step).  q and k may have fewer heads than v (qk_heads; head h
+// token's key is multiplied by dt (a discretised state-space step); 4 = one (decay, key factor) pair per head and token as given
+// by z [T, heads, 2] (a gated memory whose log weights were stabilised beforehand).  Columns of the state from v_cols up have
+// no value: v is 1 there, so that column v_cols carries the decayed sum of the keys themselves (a normaliser).  q and k may have fewer heads than v (qk_heads; head h
 // reads query/key head h / (heads / qk_heads)).  skip [heads]: o_t += skip[h] v_t.  BONUS: the read-out comes BEFORE the
 // update and sees the token's own k v^T weighted by bonus [heads, dk] instead: o_t = (S + diag(bonus) k_t v_t^T)^T q_t.
 template <typename T, int KR /* rows per lane: dk <= 4 * KR */, int kLaTokens /* tokens staged at a time */, bool BONUS>
@@ -59,11 +59,11 @@ decay_scan_kernel(const T *__restrict__ q, long long q_token, long long q_head, 
                   const int32_t *__restrict__ seq_info,
                   float *__restrict__ state, long long slot_stride, int num_slots, float *__restrict__ out, int pass, int max_segments,
                   float *__restrict__ seg_state, float *__restrict__ seg_decay, int decay_kind, const T *__restrict__ a_log,
-                  const T *__restrict__ bonus, int qk_heads, const T *__restrict__ skip) {
+                  const T *__restrict__ bonus, int qk_heads, const T *__restrict__ skip, int v_cols) {
     __shared__ float4 sx[kLaTokens * 4 * KR];  // per token and key channel: (decay, k, scaled q, -), one 16-byte read per row
     __shared__ float sv[kLaTokens * kLaCols];
     __shared__ float sprod[4 * KR];
-    __shared__ float2 s_step[kLaTokens];  // decay_kind 3: the token's (decay, step size), worked out once per token
+    __shared__ float2 s_step[kLaTokens];  // decay_kind 3, 4: the token's (decay, key factor), worked out or read once per token
     __shared__ float2 s_chan[4 * KR];     // per key channel of this head: (the decay logit's bias, the bonus), read once
     const int colblocks = (dv + kLaCols - 1) / kLaCols;
     const int s = blockIdx.x, head = blockIdx.y / colblocks, col0 = (blockIdx.y % colblocks) * kLaCols, c = blockIdx.z;
@@ -92,7 +92,7 @@ decay_scan_kernel(const T *__restrict__ q, long long q_token, long long q_head, 
     if (pass == 1)
         for (int d = threadIdx.x; d < dk; d += blockDim.x) sprod[d] = 1.f;
     for (int d = threadIdx.x; d < dk; d += blockDim.x)
-        s_chan[d] = make_float2((z_bias && decay_kind != 3) ? to_f(z_bias[(size_t)head * dk + d]) : 0.f, BONUS ? to_f(bonus[(size_t)head * dk + d]) : 0.f);
+        s_chan[d] = make_float2((z_bias && decay_kind < 3) ? to_f(z_bias[(size_t)head * dk + d]) : 0.f, BONUS ? to_f(bonus[(size_t)head * dk + d]) : 0.f);
     const int qk_head = head / (heads / qk_heads);
     const float rate = decay_kind == 3 ? expf(to_f(a_log[head])) : 0.f;
     const float skipv = skip ? to_f(skip[head]) : 0.f;
@@ -106,6 +106,9 @@ decay_scan_kernel(const T *__restrict__ q, long long q_token, long long q_head, 
                 s_step[threadIdx.x] = make_float2(expf(-rate * dt), dt);
             }
             __syncthreads();
+        } else if (decay_kind == 4) {
+            if (threadIdx.x < n) s_step[threadIdx.x] = *reinterpret_cast<const float2 *>(z + (size_t)(first + t0 + threadIdx.x) * z_token + 2 * head);
+            __syncthreads();
         }
         for (int e = threadIdx.x; e < n * dk; e += blockDim.x) {
             int j = e / dk, d = e - j * dk;
@@ -113,7 +116,7 @@ decay_scan_kernel(const T *__restrict__ q, long long q_token, long long q_head, 
             float alpha, kmul = 1.f;
             if (head_decay) alpha = head_decay[head];
             else if (decay_kind == 2) alpha = expf(-expf(z[tok * z_token + (size_t)head * dk + d] + s_chan[d].x));
-            else if (decay_kind == 3) alpha = s_step[j].x, kmul = s_step[j].y;
+            else if (decay_kind >= 3) alpha = s_step[j].x, kmul = s_step[j].y;
             else alpha = expf(log_sigmoid(z[tok * z_token + (size_t)head * dk + d] + s_chan[d].x) * inv_tau);
             const T *kp = k + tok * k_token + (size_t)qk_head * k_head, *qp = q + tok * q_token + (size_t)qk_head * q_head;
             float kd = to_f(kp[d]), qd = to_f(qp[d]);
@@ -131,7 +134,7 @@ decay_scan_kernel(const T *__restrict__ q, long long q_token, long long q_head, 
         }
         for (int e = threadIdx.x; e < n * kLaCols; e += blockDim.x) {
             int j = e / kLaCols, d = e - j * kLaCols;
-            sv[e] = col0 + d < dv ? to_f(v[(size_t)(first + t0 + j) * v_token + (size_t)head * v_head + col0 + d]) : 0.f;
+            sv[e] = col0 + d < v_cols ? to_f(v[(size_t)(first + t0 + j) * v_token + (size_t)head * v_head + col0 + d]) : col0 + d < dv ? 1.f : 0.f;
         }
         __syncthreads();
         if (pass == 1) {  // the segment's decay product per key channel, in token order
@@ -227,17 +230,20 @@ decay_combine_kernel(const int32_t *__restrict__ seq_info, const float *__restri
 
 // out[t, h, :] = o[t, h, :] / rms(o[t, h, :]) * w * act(gate[t, h, :]); one warp per (token, head).  act 0 = none, 1 = silu,
 // 2 = sigmoid; w == NULL: no weight; wide_weight: w is [heads * dv] (every head its own part) instead of [dv] shared by the
-// heads; gate_first: the gate multiplies o BEFORE the norm, out = n / rms(n) * w with n = o * act(gate).
+// heads; gate_first: the gate multiplies o BEFORE the norm, out = n / rms(n) * w with n = o * act(gate).  floor: a row of o has one
+// more column, and o is first divided by max(|that column|, floor[t, h]) + den_eps (a normalised memory's read-out).
 template <typename T>
 __global__ void __launch_bounds__(128)
 head_norm_gate_kernel(const float *__restrict__ o, const T *__restrict__ w, float eps, const T *__restrict__ gate, long long g_token, int act,
-                      T *__restrict__ out, long long rows, int heads, int dv, int wide_weight, int gate_first) {
+                      T *__restrict__ out, long long rows, int heads, int dv, int wide_weight, int gate_first, int o_row,
+                      const float *__restrict__ floor, float den_eps) {
     long long row = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (row >= rows) return;
     const int lane = threadIdx.x & 31;
     const long long t = row / heads;
     const int head = (int)(row - t * heads);
-    const float *src = o + (size_t)row * dv;
+    const float *src = o + (size_t)row * o_row;
+    const float share = floor ? 1.0f / (fmaxf(fabsf(src[dv]), floor[row]) + den_eps) : 1.f;
     auto gated = [&](int d) {
         float gv = to_f(gate[(size_t)t * g_token + (size_t)head * dv + d]);
         return act == 1 ? gv / (1.0f + expf(-gv)) : act == 2 ? 1.0f / (1.0f + expf(-gv)) : gv;
@@ -245,14 +251,14 @@ head_norm_gate_kernel(const float *__restrict__ o, const T *__restrict__ w, floa
     const bool first = gate && gate_first;
     float ss = 0.f;
     for (int d = lane; d < dv; d += 32) {
-        float x = first ? src[d] * gated(d) : src[d];
+        float x = first ? src[d] * gated(d) : src[d] * share;
         ss += x * x;
     }
     ss = warp_sum(ss);
     float inv = 1.0f / sqrtf(ss / (float)dv + eps);
     const T *wr = w ? w + (wide_weight ? (size_t)head * dv : 0) : nullptr;
     for (int d = lane; d < dv; d += 32) {
-        float y = src[d] * inv * (wr ? to_f(wr[d]) : 1.f);
+        float y = src[d] * share * inv * (wr ? to_f(wr[d]) : 1.f);
         if (gate) y *= gated(d);
         out[(size_t)row * dv + d] = from_f<T>(y);
     }
@@ -275,12 +281,14 @@ int tlb_decay_scan(const void *q, long long q_token, long long q_head, const voi
                    const float *rope_cos, const float *rope_sin, int rope_dims, int rope_interleaved, float q_scale, int heads,
                    int dk, int dv, const int32_t *seq_info, int num_seqs, int max_tokens_per_seq, float *state, long long slot_stride, int num_slots,
                    float *out, void *workspace, size_t workspace_bytes, int decay_kind, const void *a_log, const void *bonus, int qk_heads,
-                   const void *skip, int dtype, void *stream) {
+                   const void *skip, int v_cols, int dtype, void *stream) {
     if (num_seqs <= 0) return TL_OK;
     if (qk_heads <= 0) qk_heads = heads;
-    if ((decay_kind != 0 && decay_kind != 2 && decay_kind != 3) || (decay_kind != 0 && (!z || head_decay)) || (decay_kind == 3 && !a_log) ||
-        heads % qk_heads)
+    if ((decay_kind != 0 && decay_kind != 2 && decay_kind != 3 && decay_kind != 4) || (decay_kind != 0 && (!z || head_decay)) || (decay_kind == 3 && !a_log) ||
+        (decay_kind == 4 && ((uintptr_t)z % 8 || z_token % 2)) || heads % qk_heads)
         return tl::fail(TL_EINVAL, "decay_scan: bad decay kind or head groups");
+    if (v_cols <= 0) v_cols = dv;
+    if (v_cols > dv) return tl::fail(TL_EINVAL, "decay_scan: %d value columns in a state of %d", v_cols, dv);
     if (!q || !k || !v || (!z && !head_decay) || !seq_info || !state || !out || heads <= 0 || dk <= 0 || dv <= 0 || (z && !(tau > 0.f)) ||
         num_slots <= 0 || max_tokens_per_seq <= 0)
         return tl::fail(TL_EINVAL, "decay_scan: bad argument");
@@ -304,7 +312,7 @@ int tlb_decay_scan(const void *q, long long q_token, long long q_head, const voi
     decay_scan_kernel<T, KRV, (KRV > 32 ? 8 : 16), BON><<<dim3(num_seqs, heads * colblocks, GZ), kLaCols * kLaLanes, 0, st>>>(                                           \
         (const T *)q, q_token, q_head, (const T *)k, k_token, k_head, (const T *)v, v_token, v_head, z, z_token, (const T *)z_bias, z ? 1.0f / tau : 0.f, head_decay, \
         rope_cos, rope_sin, rope_dims, rope_interleaved, q_scale, heads, dk, dv, seq_info, state, slot_stride, num_slots, out, PASS, max_segments, seg_state, seg_decay, \
-        decay_kind, (const T *)a_log, (const T *)bonus, qk_heads, (const T *)skip)
+        decay_kind, (const T *)a_log, (const T *)bonus, qk_heads, (const T *)skip, v_cols)
 #define TLB_DS_K(KRV, PASS, GZ) do { if (bonus) TLB_DS_B(KRV, PASS, GZ, true); else TLB_DS_B(KRV, PASS, GZ, false); } while (0)
 #define TLB_DS(PASS, GZ) TLB_DISPATCH(dtype, "decay_scan", if (kr <= 8) TLB_DS_K(8, PASS, GZ); else if (kr <= 16) TLB_DS_K(16, PASS, GZ); else if (kr <= 32) TLB_DS_K(32, PASS, GZ); else TLB_DS_K(64, PASS, GZ))
     if (!segmented) {
@@ -326,13 +334,15 @@ int tlb_decay_scan(const void *q, long long q_token, long long q_head, const voi
 }
 
 int tlb_head_norm_gate(const float *o, const void *w, float eps, const void *gate, long long g_token, int act, void *out, int tokens, int heads,
-                       int dv, int wide_weight, int gate_first, int dtype, void *stream) {
+                       int dv, int wide_weight, int gate_first, int o_row, const float *floor, float den_eps, int dtype, void *stream) {
     if (tokens <= 0) return TL_OK;
     if (!o || !out || heads <= 0 || dv <= 0 || act < 0 || act > 2) return tl::fail(TL_EINVAL, "head_norm_gate: bad argument");
+    if (o_row <= 0) o_row = dv;
+    if (o_row < dv + (floor ? 1 : 0) || (floor && gate_first)) return tl::fail(TL_EINVAL, "head_norm_gate: bad row or normaliser");
     long long rows = (long long)tokens * heads;
     TLB_DISPATCH(dtype, "head_norm_gate",
                  head_norm_gate_kernel<T><<<(unsigned)((rows + 3) / 4), 128, 0, as_stream(stream)>>>(o, (const T *)w, eps, (const T *)gate, g_token, act,
-                                                                                                    (T *)out, rows, heads, dv, wide_weight, gate_first));
+                                                                                                    (T *)out, rows, heads, dv, wide_weight, gate_first, o_row, floor, den_eps));
     TL_LAUNCH_CHECK("head_norm_gate");
     return TL_OK;
 }

@@ -12,10 +12,7 @@ namespace tlb {
 constexpr int kTileRows = TLB_MOE_TILE_ROWS;
 
 __device__ __forceinline__ float moe_act(float z, int act) {
-    if (act == 0) return z / (1.0f + expf(-z));
-    if (act == 2) return z > 0.f ? z * z : 0.f;  // squared ReLU
-    float inner = 0.7978845608028654f * (z + 0.044715f * z * z * z);
-    return 0.5f * z * (1.0f + tanhf(inner));
+    return act == 2 ? (z > 0.f ? z * z : 0.f) : act_apply(z, act);  // 2: squared ReLU
 }
 
 // Which rows of `a` a tile's rows read: the sorted rows themselves (the second product), the token of the pair, or the pair.
@@ -25,26 +22,31 @@ __device__ __forceinline__ int moe_src_row(int pair, int sorted_row, int top, in
     return gather == kGatherSorted ? sorted_row : gather == kGatherToken ? pair / top : pair;
 }
 
+// aux_w: one more row of weights that is no router output; aux[t] = sigmoid(aux_w . h_t) (the gate of a shared expert).
 // One CTA per token: the row of h is staged in shared memory as fp32, the warps share the experts (each logit is one
 // warp's dot product in a fixed lane order, so it does not depend on the launch), then warp 0 picks the top-k.
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_route_kernel(const T *__restrict__ h, const T *__restrict__ w, const T *__restrict__ b, int tokens, int dim, int experts, int top, int scoring,
-                 const T *__restrict__ choice_bias, float weight_scale, int32_t *__restrict__ idx, float *__restrict__ gate) {
+                 const T *__restrict__ choice_bias, float weight_scale, int group_count, int group_keep, const T *__restrict__ aux_w,
+                 float *__restrict__ aux, int32_t *__restrict__ idx, float *__restrict__ gate) {
     extern __shared__ float route_smem[];
     float *x = route_smem;        // [dim]
     float *z = route_smem + dim;  // [experts]: what the choice is made by
     float *p_all = z + experts;   // [experts]: scoring 2, the softmax over all outputs
+    float *best = p_all + experts;  // [group_count]: the largest choice score of every group
     const int t = blockIdx.x;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
     for (int d = threadIdx.x; d < dim; d += blockDim.x) x[d] = to_f(h[(size_t)t * dim + d]);
     __syncthreads();
-    for (int e = warp; e < experts; e += warps) {
-        const T *row = w + (size_t)e * dim;
+    for (int e = warp; e < experts + (aux_w ? 1 : 0); e += warps) {
+        const T *row = e < experts ? w + (size_t)e * dim : aux_w;
         float s = 0.f;
         for (int d = lane; d < dim; d += 32) s = fmaf(x[d], to_f(row[d]), s);
         s = warp_sum(s);
-        if (lane == 0) z[e] = s + (b ? to_f(b[e]) : 0.f);
+        if (lane != 0) continue;
+        if (e < experts) z[e] = s + (b ? to_f(b[e]) : 0.f);
+        else aux[t] = sigmoid(s);
     }
     __syncthreads();
     if (warp != 0) return;
@@ -58,6 +60,22 @@ moe_route_kernel(const T *__restrict__ h, const T *__restrict__ w, const T *__re
             float p = expf(z[e] - m) / sum;
             p_all[e] = p;
             z[e] = p + (choice_bias ? to_f(choice_bias[e]) : 0.f);
+        }
+        __syncwarp();
+    }
+    if (group_keep > 0 && group_keep < group_count) {  // only the outputs of the best groups of neighbours can be chosen
+        const int size = experts / group_count;
+        for (int j = lane; j < group_count; j += 32) {
+            float m = -INFINITY;
+            for (int e = j * size; e < (j + 1) * size; ++e) m = fmaxf(m, z[e]);
+            best[j] = m;
+        }
+        __syncwarp();
+        for (int e = lane; e < experts; e += 32) {
+            const int j = e / size;
+            int ahead = 0;  // groups in front of this one (lower index wins a tie)
+            for (int i = 0; i < group_count; ++i) ahead += best[i] > best[j] || (best[i] == best[j] && i < j);
+            if (ahead >= group_keep) z[e] = -INFINITY;
         }
         __syncwarp();
     }
@@ -130,8 +148,8 @@ constexpr int kBN = 64, kBK = 16;
 template <typename T, bool GATED>
 __global__ void __launch_bounds__(256)
 moe_grouped_kernel(const T *__restrict__ a, const T *__restrict__ w1, const T *__restrict__ w2, const int32_t *__restrict__ sorted_pair,
-                   const int32_t *__restrict__ tile_expert, const int32_t *__restrict__ counters, int top, int K, int N, int act, int gather,
-                   T *__restrict__ inter, float *__restrict__ pair_out) {
+                   const int32_t *__restrict__ tile_expert, const int32_t *__restrict__ counters, int top, int K, int N, int act, float limit, float slope,
+                   int gather, T *__restrict__ inter, float *__restrict__ pair_out) {
     if ((int)blockIdx.x >= counters[0]) return;
     __shared__ float sa[kBK][kTileRows + 1];
     __shared__ float sb1[kBK][kBN + 1];
@@ -187,7 +205,7 @@ moe_grouped_kernel(const T *__restrict__ a, const T *__restrict__ w1, const T *_
         for (int c = 0; c < 4; ++c) {
             int col = col0 + tx + 16 * c;
             if (col >= N) continue;
-            if (GATED) inter[(size_t)row * N + col] = from_f<T>(moe_act(c1[r][c], act) * c2[r][c]);
+            if (GATED) inter[(size_t)row * N + col] = from_f<T>(gated_pair(c1[r][c], c2[r][c], act, limit, slope));
             else if (inter) inter[(size_t)row * N + col] = from_f<T>(moe_act(c1[r][c], act));
             else pair_out[(size_t)pair * N + col] = c1[r][c];
         }
@@ -219,8 +237,8 @@ __device__ __forceinline__ void moe_cp16(void *dst, const void *src, bool ok) {
 template <bool GATED, int BM>
 __global__ void __launch_bounds__(256)
 moe_grouped_mma_kernel(const bf16 *__restrict__ a, const bf16 *__restrict__ w1, const bf16 *__restrict__ w2, const int32_t *__restrict__ sorted_pair,
-                       const int32_t *__restrict__ tile_expert, const int32_t *__restrict__ counters, int top, int K, int N, int act, int gather,
-                       bf16 *__restrict__ inter, float *__restrict__ pair_out) {
+                       const int32_t *__restrict__ tile_expert, const int32_t *__restrict__ counters, int top, int K, int N, int act, float limit,
+                       float slope, int gather, bf16 *__restrict__ inter, float *__restrict__ pair_out) {
     if ((int)blockIdx.x >= counters[0]) return;
     constexpr int MT = BM / 16;          // 16-row halves/quarters of the tile
     constexpr int NW = 8 / MT;           // warps along the columns
@@ -301,7 +319,7 @@ moe_grouped_mma_kernel(const bf16 *__restrict__ a, const bf16 *__restrict__ w1, 
                 int col = col0 + nq * (8 * NPW) + i * 8 + 2 * t + j;
                 if (col >= N) continue;
                 float v = c1[i][half * 2 + j];
-                if (GATED) inter[(size_t)row * N + col] = __float2bfloat16_rn(moe_act(v, act) * c2[i][half * 2 + j]);
+                if (GATED) inter[(size_t)row * N + col] = __float2bfloat16_rn(gated_pair(v, c2[i][half * 2 + j], act, limit, slope));
                 else if (inter) inter[(size_t)row * N + col] = __float2bfloat16_rn(moe_act(v, act));
                 else pair_out[(size_t)pair * N + col] = v;
             }
@@ -321,7 +339,7 @@ __global__ void moe_scale_rows_kernel(const T *__restrict__ h, const float *__re
 // idx != NULL: a choice whose expert id is >= experts is an identity expert, its output the token's input row h[t, :].
 template <typename T>
 __global__ void moe_combine_kernel(const float *__restrict__ pair_out, const float *__restrict__ gate, const T *__restrict__ shared,
-                                   const int32_t *__restrict__ idx, int experts, const T *__restrict__ h, float *__restrict__ y, int top, int dim) {
+                                   const float *__restrict__ shared_gate, const int32_t *__restrict__ idx, int experts, const T *__restrict__ h, float *__restrict__ y, int top, int dim) {
     int t = blockIdx.x;
     for (int d = threadIdx.x; d < dim; d += blockDim.x) {
         float s = 0.f;
@@ -329,7 +347,7 @@ __global__ void moe_combine_kernel(const float *__restrict__ pair_out, const flo
             const bool same = idx != nullptr && idx[(size_t)t * top + k] >= experts;
             s = fmaf(gate ? gate[(size_t)t * top + k] : 1.f, same ? to_f(h[(size_t)t * dim + d]) : pair_out[((size_t)t * top + k) * dim + d], s);
         }
-        if (shared) s += to_f(shared[(size_t)t * dim + d]);
+        if (shared) s = fmaf(shared_gate ? shared_gate[t] : 1.f, to_f(shared[(size_t)t * dim + d]), s);
         y[(size_t)t * dim + d] = s;
     }
 }
@@ -340,7 +358,7 @@ using namespace tlb;
 
 template <bool GATED, int BM>
 static int launch_grouped_mma(dim3 grid, cudaStream_t st, const bf16 *a, const bf16 *w1, const bf16 *w2, const int32_t *sorted_pair,
-                              const int32_t *tile_expert, const int32_t *counters, int top, int K, int N, int act, int gather, bf16 *inter,
+                              const int32_t *tile_expert, const int32_t *counters, int top, int K, int N, int act, float limit, float slope, int gather, bf16 *inter,
                               float *pair_out) {
     size_t smem = (size_t)2 * (BM + kTN * (GATED ? 2 : 1)) * kTS * sizeof(bf16);
     auto kernel = moe_grouped_mma_kernel<GATED, BM>;
@@ -348,7 +366,7 @@ static int launch_grouped_mma(dim3 grid, cudaStream_t st, const bf16 *a, const b
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return tl::fail(TL_ECUDA, "moe_grouped: %s", cudaGetErrorString(e));
     }
-    kernel<<<grid, 256, smem, st>>>(a, w1, w2, sorted_pair, tile_expert, counters, top, K, N, act, gather, inter, pair_out);
+    kernel<<<grid, 256, smem, st>>>(a, w1, w2, sorted_pair, tile_expert, counters, top, K, N, act, limit, slope, gather, inter, pair_out);
     return TL_OK;
 }
 
@@ -359,15 +377,19 @@ static bool moe_mma_ok(int dtype, int k, const void *a, const void *w1, const vo
 extern "C" {
 
 int tlb_moe_route(const void *h, const void *w, const void *b, int tokens, int dim, int experts, int top, int scoring, const void *choice_bias,
-                  float weight_scale, int32_t *idx, float *gate, int dtype, void *stream) {
+                  float weight_scale, int group_count, int group_keep, const void *aux_w, float *aux, int32_t *idx, float *gate, int dtype, void *stream) {
     if (tokens <= 0) return TL_OK;
     if (!h || !w || !idx || !gate || dim <= 0 || experts <= 0 || top <= 0 || top > experts || scoring < 0 || scoring > 2)
         return tl::fail(TL_EINVAL, "moe_route: bad argument");
-    size_t smem = ((size_t)dim + 2 * (size_t)experts) * sizeof(float);
+    if ((aux_w == nullptr) != (aux == nullptr) || group_count < 0 || group_keep < 0 || group_keep > group_count ||
+        (group_count > 0 && (experts % group_count || group_keep * (experts / group_count) < top)))
+        return tl::fail(TL_EINVAL, "moe_route: bad groups or side output");
+    size_t smem = ((size_t)dim + 2 * (size_t)experts + group_count) * sizeof(float);
     if (smem > 48 * 1024) return tl::fail(TL_EINVAL, "moe_route: width %d + %d experts do not fit", dim, experts);
     TLB_DISPATCH(dtype, "moe_route",
                  moe_route_kernel<T><<<tokens, 256, smem, as_stream(stream)>>>((const T *)h, (const T *)w, (const T *)b, tokens, dim, experts, top, scoring,
-                                                                             (const T *)choice_bias, weight_scale, idx, gate));
+                                                                             (const T *)choice_bias, weight_scale, group_count, group_keep, (const T *)aux_w, aux,
+                                                                             idx, gate));
     TL_LAUNCH_CHECK("moe_route");
     return TL_OK;
 }
@@ -395,16 +417,17 @@ int tlb_moe_sort(const int32_t *idx, int tokens, int top, int experts, int tile_
 // The tensor-core kernels take 32- or 64-row expert tiles (64 halves the weight traffic per row when experts get many
 // rows); the fp32 kernels 32 only.
 int tlb_moe_gate_up(const void *h, const void *wg, const void *wu, const int32_t *sorted_pair, const int32_t *tile_expert, const int32_t *counters,
-                    int tokens, int top, int experts, int tile_rows, int dim, int ff, int act, void *inter, int dtype, void *stream) {
+                    int tokens, int top, int experts, int tile_rows, int dim, int ff, int act, float limit, float slope, void *inter, int dtype, void *stream) {
     if (tokens <= 0) return TL_OK;
-    if (!h || !wg || !wu || !sorted_pair || !tile_expert || !counters || !inter || dim <= 0 || ff <= 0 || top <= 0)
+    if (!h || !wg || !wu || !sorted_pair || !tile_expert || !counters || !inter || dim <= 0 || ff <= 0 || top <= 0 || (act != 0 && act != 1 && act != 3) ||
+        (act == 3 && !(limit > 0.f)))
         return tl::fail(TL_EINVAL, "moe_gate_up: bad argument");
     if (moe_mma_ok(dtype, dim, h, wg, wu)) {
         dim3 tc((unsigned)(tlb_moe_max_rows(tokens, top, experts, tile_rows) / tile_rows), ceil_div(ff, kTN));
         int rc = tile_rows == 64 ? launch_grouped_mma<true, 64>(tc, as_stream(stream), (const bf16 *)h, (const bf16 *)wg, (const bf16 *)wu, sorted_pair,
-                                                                tile_expert, counters, top, dim, ff, act, kGatherToken, (bf16 *)inter, nullptr)
+                                                                tile_expert, counters, top, dim, ff, act, limit, slope, kGatherToken, (bf16 *)inter, nullptr)
                                  : launch_grouped_mma<true, 32>(tc, as_stream(stream), (const bf16 *)h, (const bf16 *)wg, (const bf16 *)wu, sorted_pair,
-                                                                tile_expert, counters, top, dim, ff, act, kGatherToken, (bf16 *)inter, nullptr);
+                                                                tile_expert, counters, top, dim, ff, act, limit, slope, kGatherToken, (bf16 *)inter, nullptr);
         if (rc != TL_OK) return rc;
         TL_LAUNCH_CHECK("moe_gate_up");
         return TL_OK;
@@ -413,7 +436,7 @@ int tlb_moe_gate_up(const void *h, const void *wg, const void *wu, const int32_t
     dim3 grid((unsigned)(tlb_moe_max_rows(tokens, top, experts, kTileRows) / kTileRows), ceil_div(ff, kBN));
     TLB_DISPATCH(dtype, "moe_gate_up",
                  moe_grouped_kernel<T, true><<<grid, 256, 0, as_stream(stream)>>>((const T *)h, (const T *)wg, (const T *)wu, sorted_pair, tile_expert,
-                                                                                 counters, top, dim, ff, act, kGatherToken, (T *)inter, nullptr));
+                                                                                 counters, top, dim, ff, act, limit, slope, kGatherToken, (T *)inter, nullptr));
     TL_LAUNCH_CHECK("moe_gate_up");
     return TL_OK;
 }
@@ -429,9 +452,9 @@ int tlb_moe_up(const void *a, const void *wu, const int32_t *sorted_pair, const 
     if (moe_mma_ok(dtype, dim, a, wu, nullptr)) {
         dim3 tc((unsigned)(tlb_moe_max_rows(tokens, top, experts, tile_rows) / tile_rows), ceil_div(ff, kTN));
         int rc = tile_rows == 64 ? launch_grouped_mma<false, 64>(tc, as_stream(stream), (const bf16 *)a, (const bf16 *)wu, nullptr, sorted_pair, tile_expert,
-                                                                 counters, top, dim, ff, act, gather, (bf16 *)inter, nullptr)
+                                                                 counters, top, dim, ff, act, 0.f, 1.f, gather, (bf16 *)inter, nullptr)
                                  : launch_grouped_mma<false, 32>(tc, as_stream(stream), (const bf16 *)a, (const bf16 *)wu, nullptr, sorted_pair, tile_expert,
-                                                                 counters, top, dim, ff, act, gather, (bf16 *)inter, nullptr);
+                                                                 counters, top, dim, ff, act, 0.f, 1.f, gather, (bf16 *)inter, nullptr);
         if (rc != TL_OK) return rc;
         TL_LAUNCH_CHECK("moe_up");
         return TL_OK;
@@ -440,7 +463,7 @@ int tlb_moe_up(const void *a, const void *wu, const int32_t *sorted_pair, const 
     dim3 grid((unsigned)(tlb_moe_max_rows(tokens, top, experts, kTileRows) / kTileRows), ceil_div(ff, kBN));
     TLB_DISPATCH(dtype, "moe_up",
                  moe_grouped_kernel<T, false><<<grid, 256, 0, as_stream(stream)>>>((const T *)a, (const T *)wu, nullptr, sorted_pair, tile_expert, counters,
-                                                                                  top, dim, ff, act, gather, (T *)inter, nullptr));
+                                                                                  top, dim, ff, act, 0.f, 1.f, gather, (T *)inter, nullptr));
     TL_LAUNCH_CHECK("moe_up");
     return TL_OK;
 }
@@ -462,9 +485,9 @@ int tlb_moe_down(const void *inter, const void *wd, const int32_t *sorted_pair, 
     if (moe_mma_ok(dtype, ff, inter, wd, nullptr)) {
         dim3 tc((unsigned)(tlb_moe_max_rows(tokens, top, experts, tile_rows) / tile_rows), ceil_div(dim, kTN));
         int rc = tile_rows == 64 ? launch_grouped_mma<false, 64>(tc, as_stream(stream), (const bf16 *)inter, (const bf16 *)wd, nullptr, sorted_pair,
-                                                                 tile_expert, counters, top, ff, dim, 0, kGatherSorted, nullptr, pair_out)
+                                                                 tile_expert, counters, top, ff, dim, 0, 0.f, 1.f, kGatherSorted, nullptr, pair_out)
                                  : launch_grouped_mma<false, 32>(tc, as_stream(stream), (const bf16 *)inter, (const bf16 *)wd, nullptr, sorted_pair,
-                                                                 tile_expert, counters, top, ff, dim, 0, kGatherSorted, nullptr, pair_out);
+                                                                 tile_expert, counters, top, ff, dim, 0, 0.f, 1.f, kGatherSorted, nullptr, pair_out);
         if (rc != TL_OK) return rc;
         TL_LAUNCH_CHECK("moe_down");
         return TL_OK;
@@ -473,17 +496,17 @@ int tlb_moe_down(const void *inter, const void *wd, const int32_t *sorted_pair, 
     dim3 grid((unsigned)(tlb_moe_max_rows(tokens, top, experts, kTileRows) / kTileRows), ceil_div(dim, kBN));
     TLB_DISPATCH(dtype, "moe_down",
                  moe_grouped_kernel<T, false><<<grid, 256, 0, as_stream(stream)>>>((const T *)inter, (const T *)wd, nullptr, sorted_pair, tile_expert,
-                                                                                  counters, top, ff, dim, 0, kGatherSorted, nullptr, pair_out));
+                                                                                  counters, top, ff, dim, 0, 0.f, 1.f, kGatherSorted, nullptr, pair_out));
     TL_LAUNCH_CHECK("moe_down");
     return TL_OK;
 }
 
-int tlb_moe_combine(const float *pair_out, const float *gate, const void *shared, const int32_t *idx, int experts, const void *h, float *y, int tokens,
+int tlb_moe_combine(const float *pair_out, const float *gate, const void *shared, const float *shared_gate, const int32_t *idx, int experts, const void *h, float *y, int tokens,
                     int top, int dim, int dtype, void *stream) {
     if (tokens <= 0) return TL_OK;
     if (!pair_out || !y || top <= 0 || dim <= 0 || (idx && !h)) return tl::fail(TL_EINVAL, "moe_combine: bad argument");
     TLB_DISPATCH(dtype, "moe_combine",
-                 moe_combine_kernel<T><<<tokens, 256, 0, as_stream(stream)>>>(pair_out, gate, (const T *)shared, idx, experts, (const T *)h, y, top, dim));
+                 moe_combine_kernel<T><<<tokens, 256, 0, as_stream(stream)>>>(pair_out, gate, (const T *)shared, shared_gate, idx, experts, (const T *)h, y, top, dim));
     TL_LAUNCH_CHECK("moe_combine");
     return TL_OK;
 }

@@ -10,7 +10,7 @@
 //   mask 2  the earlier positions of its own block of `size` positions, blocks counted from position 0 (chunks)
 // and so are a tanh soft cap on the scaled scores, a sink (one more term in the softmax's denominator that carries no
 // value: exp(0), or exp(head_bias[h]) with a learned number per head) and a per-head output gate (the output of head h
-// times sigmoid(gate[t, h])).  weights 1 replaces the softmax: a visible key weighs sigmoid(score + head_bias[h]) and
+// times sigmoid(gate[t, h]); gate_wide: entry d of head h times sigmoid(gate[t, h * dv + d])).  weights 1 replaces the softmax: a visible key weighs sigmoid(score + head_bias[h]) and
 // nothing is normalised over the keys.
 // Scores, the running maximum / sum and the accumulators are fp32; cache rows are converted as they are staged, so the
 // same kernel serves the bf16 and the fp32 cache.  Key tiles are 32-aligned in absolute positions and taken in
@@ -38,7 +38,7 @@ __global__ void __launch_bounds__(kPaWarps * 32)
 paged_attention_kernel(const T *__restrict__ q, long long q_token, long long q_head, const T *__restrict__ slab, int num_pages, int page_size,
                        int row_width, int dk, int dv, int heads, int kv_heads, const int32_t *__restrict__ block_table, int max_pages,
                        const int32_t *__restrict__ tiles, const int32_t *__restrict__ tok_pos, int mask, int mask_size, int keep_first, float scale, float softcap,
-                       int sink, const T *__restrict__ gate, long long g_token, T *__restrict__ out, long long o_token, long long o_head,
+                       int sink, const T *__restrict__ gate, long long g_token, int gate_wide, T *__restrict__ out, long long o_token, long long o_head,
                        const float *__restrict__ head_bias, int weights) {
     extern __shared__ float smem[];
     const int kstride = dk + 1;            // +1 breaks the bank conflict of lane = key reads
@@ -147,11 +147,13 @@ paged_attention_kernel(const T *__restrict__ q, long long q_token, long long q_h
     auto finish = [&](int r, int tq, float l, const float *acc) {
         int head = head0 + r % hp;
         float inv = 1.0f / l;
-        if (gate) inv *= 1.0f / (1.0f + expf(-to_f(gate[(size_t)(first + tq) * g_token + head])));
+        if (gate && !gate_wide) inv *= sigmoid(to_f(gate[(size_t)(first + tq) * g_token + head]));
+        const T *gw = gate && gate_wide ? gate + (size_t)(first + tq) * g_token + (size_t)head * dv : nullptr;
         T *o = out + (size_t)(first + tq) * o_token + (size_t)head * o_head;
 #pragma unroll
         for (int i = 0; i < VL; ++i)
-            if (lane + 32 * i < dv) o[lane + 32 * i] = from_f<T>(acc[i] * inv);
+            if (lane + 32 * i < dv)
+                o[lane + 32 * i] = from_f<T>(acc[i] * (gw ? inv * sigmoid(to_f(gw[lane + 32 * i])) : inv));
     };
     if (live0) finish(r0, tq0, l0, acc0);
     if (live1) finish(r1, tq1, l1, acc1);
@@ -414,7 +416,7 @@ qk_whole_prepare_wide_kernel(bf16 *q, long long q_token, int heads, const bf16 *
 template <typename T, int VL>
 static int pa_launch(const void *q, long long q_token, long long q_head, const void *slab, int num_pages, int page_size, int dk, int dv, int heads,
                      int kv_heads, const int32_t *block_table, int max_pages, const int32_t *tiles, int num_tiles, const int32_t *tok_pos, int mask,
-                     int mask_size, int keep_first, float scale, float softcap, int sink, const void *gate, long long g_token, void *out, long long o_token,
+                     int mask_size, int keep_first, float scale, float softcap, int sink, const void *gate, long long g_token, int gate_wide, void *out, long long o_token,
                      long long o_head, const float *head_bias, int weights, cudaStream_t st) {
     size_t smem = ((size_t)kPaRows * dk + (size_t)kPaKeys * (dk + 1) + (size_t)kPaKeys * dv) * sizeof(float);
     auto kernel = paged_attention_kernel<T, VL>;
@@ -427,7 +429,7 @@ static int pa_launch(const void *q, long long q_token, long long q_head, const v
     dim3 grid(num_tiles, kv_heads * ceil_div(group, pa_heads_per_cta(group)));
     kernel<<<grid, kPaWarps * 32, smem, st>>>((const T *)q, q_token, q_head, (const T *)slab, num_pages, page_size, kv_heads * (dk + dv), dk, dv, heads,
                                               kv_heads, block_table, max_pages, tiles, tok_pos, mask, mask_size, keep_first, scale, softcap, sink, (const T *)gate,
-                                              g_token, (T *)out, o_token, o_head, head_bias, weights);
+                                              g_token, gate_wide, (T *)out, o_token, o_head, head_bias, weights);
     return TL_OK;
 }
 
@@ -444,7 +446,7 @@ int tlb_paged_attention_tile_tokens(int heads, int kv_heads) {
 
 int tlb_paged_attention(const void *q, long long q_token, long long q_head, const void *slab, int num_pages, int page_size, int dk, int dv, int heads,
                         int kv_heads, const int32_t *block_table, int max_pages, const int32_t *tiles, int num_tiles, const int32_t *tok_pos, int mask,
-                        int mask_size, int keep_first, float scale, float softcap, int sink, const void *gate, long long g_token, void *out, long long o_token,
+                        int mask_size, int keep_first, float scale, float softcap, int sink, const void *gate, long long g_token, int gate_wide, void *out, long long o_token,
                         long long o_head, const float *head_bias, int weights, int dtype, void *stream) {
     if (num_tiles <= 0) return TL_OK;
     if (weights < 0 || weights > 1 || (weights == 1 && (sink || softcap > 0.f))) return tl::fail(TL_EINVAL, "paged_attention: bad weights mode");
@@ -460,7 +462,7 @@ int tlb_paged_attention(const void *q, long long q_token, long long q_head, cons
     int rc = TL_OK;
 #define TLB_PA(V)                                                                                                                                   \
     rc = pa_launch<T, V>(q, q_token, q_head, slab, num_pages, page_size, dk, dv, heads, kv_heads, block_table, max_pages, tiles, num_tiles, tok_pos, \
-                         mask, mask_size, keep_first, scale, softcap, sink, gate, g_token, out, o_token, o_head, head_bias, weights, st)
+                         mask, mask_size, keep_first, scale, softcap, sink, gate, g_token, gate_wide, out, o_token, o_head, head_bias, weights, st)
     TLB_DISPATCH(dtype, "paged_attention", if (vl <= 1) TLB_PA(1); else if (vl <= 2) TLB_PA(2); else if (vl <= 4) TLB_PA(4); else if (vl <= 8) TLB_PA(8);
                  else TLB_PA(16));
 #undef TLB_PA

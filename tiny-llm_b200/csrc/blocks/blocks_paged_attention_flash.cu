@@ -40,7 +40,8 @@ struct FlashArgs {
     int mask, mask_size, keep_first;
     float scale, softcap;
     int sink;
-    const bf16 *gate;
+    const bf16 *gate;   // logits of a sigmoid: one per head, or (gate_wide) one per entry of every head
+    int gate_wide;
     long long g_token;
     bf16 *out;
     long long o_token, o_head;
@@ -314,11 +315,15 @@ paged_attention_flash_kernel(const FlashArgs A) {
     auto factor = [&](int r, float sum) {  // what a row's sums are multiplied by on their way out
         const int tq = r / hp, hh = r - tq * hp;
         float inv = 1.0f / sum;
-        if (A.gate) inv *= 1.0f / (1.0f + expf(-__bfloat162float(A.gate[(size_t)(first + tq) * A.g_token + head0 + hh])));
+        if (A.gate && !A.gate_wide) inv *= sigmoid(__bfloat162float(A.gate[(size_t)(first + tq) * A.g_token + head0 + hh]));
         return inv;
     };
     auto put2 = [&](int r, int col, float x, float y) {
         const int tq = r / hp, hh = r - tq * hp;
+        if (A.gate_wide) {
+            const bf16 *gw = A.gate + (size_t)(first + tq) * A.g_token + (size_t)(head0 + hh) * A.dv + col;
+            x *= sigmoid(__bfloat162float(gw[0])), y *= sigmoid(__bfloat162float(gw[1]));
+        }
         bf16 *o = A.out + (size_t)(first + tq) * A.o_token + (size_t)(head0 + hh) * A.o_head + col;
         if (A.o_pairs) *reinterpret_cast<uint32_t *>(o) = tl::pack2<bf16>(x, y);
         else o[0] = __float2bfloat16_rn(x), o[1] = __float2bfloat16_rn(y);
@@ -436,7 +441,7 @@ int tlb_paged_attention_flash_supported(int dk, int dv, int kv_heads, int page_s
 
 int tlb_paged_attention_flash(const void *q, long long q_token, long long q_head, const void *slab, int num_pages, int page_size, int dk, int dv, int heads,
                               int kv_heads, const int32_t *block_table, int max_pages, const int32_t *tiles, int num_tiles, const int32_t *tok_pos,
-                              int mask, int mask_size, int keep_first, float scale, float softcap, int sink, const void *gate, long long g_token, void *out,
+                              int mask, int mask_size, int keep_first, float scale, float softcap, int sink, const void *gate, long long g_token, int gate_wide, void *out,
                               long long o_token, long long o_head, int split_keys, int splits, const float *head_bias, int weights, void *stream) {
     if (num_tiles <= 0) return TL_OK;
     if (weights < 0 || weights > 1 || (weights == 1 && (sink || softcap > 0.f))) return tl::fail(TL_EINVAL, "paged_attention_flash: bad weights mode");
@@ -455,7 +460,7 @@ int tlb_paged_attention_flash(const void *q, long long q_token, long long q_head
     a.dk = dk, a.dv = dv, a.heads = heads, a.kv_heads = kv_heads, a.hp = group < rows ? group : rows;
     a.block_table = block_table, a.max_pages = max_pages, a.tiles = tiles, a.tok_pos = tok_pos;
     a.mask = mask, a.mask_size = mask_size, a.keep_first = keep_first, a.scale = scale, a.softcap = softcap, a.sink = sink;
-    a.gate = (const bf16 *)gate, a.g_token = g_token, a.out = (bf16 *)out, a.o_token = o_token, a.o_head = o_head, a.head_bias = head_bias, a.weights = weights;
+    a.gate = (const bf16 *)gate, a.gate_wide = gate && gate_wide, a.g_token = g_token, a.out = (bf16 *)out, a.o_token = o_token, a.o_head = o_head, a.head_bias = head_bias, a.weights = weights;
     a.k_stride = ceil_div(dk, 16) * 16 + 8;  // (stride / 8) odd: conflict-free ldmatrix rows
     a.q_wide = tl::aligned16(q) && q_token % 8 == 0 && q_head % 8 == 0;
     a.o_pairs = (uintptr_t)out % 4 == 0 && o_token % 2 == 0 && o_head % 2 == 0;

@@ -61,7 +61,7 @@ __global__ void __launch_bounds__(kGWarps * 32)
 paged_attention_mma_kernel(const bf16 *__restrict__ q, long long q_token, long long q_head, const bf16 *__restrict__ slab, int num_pages, int page_size,
                            int row_width, int dk, int dv, int heads, int kv_heads, int hp /* query heads per CTA */,
                            const int32_t *__restrict__ block_table, int max_pages, const int32_t *__restrict__ tiles, const int32_t *__restrict__ tok_pos,
-                           int mask, int mask_size, int keep_first, float scale, float softcap, int sink, const bf16 *__restrict__ gate, long long g_token,
+                           int mask, int mask_size, int keep_first, float scale, float softcap, int sink, const bf16 *__restrict__ gate, long long g_token, int gate_wide,
                            bf16 *__restrict__ out, long long o_token, long long o_head, int k_stride, int v_stride /* shared-memory row strides */,
                            float *__restrict__ partial /* split results, or NULL */, const float *__restrict__ head_bias /* [heads] or NULL */,
                            int weights /* 0 softmax, 1 sigmoid(score + head_bias) without normalisation */) {
@@ -283,13 +283,15 @@ paged_attention_mma_kernel(const bf16 *__restrict__ q, long long q_token, long l
             if (tq >= count || hh >= nheads) continue;
             int head = head0 + hh;
             float inv = 1.0f / s_l[r];
-            if (gate) inv *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)(first + tq) * g_token + head])));
+            if (gate && !gate_wide) inv *= sigmoid(__bfloat162float(gate[(size_t)(first + tq) * g_token + head]));
+            const bf16 *gw = gate && gate_wide ? gate + (size_t)(first + tq) * g_token + (size_t)head * dv : nullptr;
             bf16 *o = out + (size_t)(first + tq) * o_token + (size_t)head * o_head;
 #pragma unroll
             for (int i = 0; i < 2 * PAIRS; ++i) {
                 int col = nt * (16 * PAIRS) + i * 8 + 2 * t;
-                if (col < dv) o[col] = __float2bfloat16_rn(acc[i][half * 2] * inv);
-                if (col + 1 < dv) o[col + 1] = __float2bfloat16_rn(acc[i][half * 2 + 1] * inv);
+                auto part_gate = [&](int c) { return gw ? inv * sigmoid(__bfloat162float(gw[c])) : inv; };
+                if (col < dv) o[col] = __float2bfloat16_rn(acc[i][half * 2] * part_gate(col));
+                if (col + 1 < dv) o[col + 1] = __float2bfloat16_rn(acc[i][half * 2 + 1] * part_gate(col + 1));
             }
         }
     }
@@ -298,7 +300,7 @@ paged_attention_mma_kernel(const bf16 *__restrict__ q, long long q_token, long l
 // Combine the split results of one query row per CTA: weights exp(m_z - max m), added in split order; then the gate.
 __global__ void __launch_bounds__(128)
 paged_attention_merge_kernel(const float *__restrict__ part, int splits, int cols, const int32_t *__restrict__ tiles, int heads, int kv_heads, int hp,
-                             int dv, const bf16 *__restrict__ gate, long long g_token, bf16 *__restrict__ out, long long o_token, long long o_head) {
+                             int dv, const bf16 *__restrict__ gate, long long g_token, int gate_wide, bf16 *__restrict__ out, long long o_token, long long o_head) {
     __shared__ float weight[64];
     __shared__ float inv_l;
     const int group = heads / kv_heads, parts = (group + hp - 1) / hp;
@@ -323,7 +325,7 @@ paged_attention_merge_kernel(const float *__restrict__ part, int splits, int col
         l = warp_sum(l);
         if (threadIdx.x == 0) {
             float inv = 1.0f / l;
-            if (gate) inv *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)(first + tq) * g_token + head0 + hh])));
+            if (gate && !gate_wide) inv *= sigmoid(__bfloat162float(gate[(size_t)(first + tq) * g_token + head0 + hh]));
             inv_l = inv;
         }
     }
@@ -332,6 +334,7 @@ paged_attention_merge_kernel(const float *__restrict__ part, int splits, int col
     for (int c = threadIdx.x; c < dv; c += blockDim.x) {
         float v = 0.f;
         for (int z = 0; z < splits; ++z) v = fmaf(base[z * step + c], weight[z], v);
+        if (gate && gate_wide) v *= sigmoid(__bfloat162float(gate[(size_t)(first + tq) * g_token + (size_t)(head0 + hh) * dv + c]));
         o[c] = __float2bfloat16_rn(v * inv_l);
     }
 }
@@ -367,7 +370,7 @@ size_t tlb_paged_attention_mma_workspace(int num_tiles, int heads, int kv_heads,
 
 int tlb_paged_attention_mma(const void *q, long long q_token, long long q_head, const void *slab, int num_pages, int page_size, int dk, int dv, int heads,
                             int kv_heads, const int32_t *block_table, int max_pages, const int32_t *tiles, int num_tiles, const int32_t *tok_pos,
-                            int mask, int mask_size, int keep_first, float scale, float softcap, int sink, const void *gate, long long g_token, void *out,
+                            int mask, int mask_size, int keep_first, float scale, float softcap, int sink, const void *gate, long long g_token, int gate_wide, void *out,
                             long long o_token, long long o_head, int splits, void *workspace, size_t workspace_bytes, const float *head_bias,
                             int weights, void *stream) {
     if (num_tiles <= 0) return TL_OK;
@@ -401,7 +404,7 @@ int tlb_paged_attention_mma(const void *q, long long q_token, long long q_head, 
         }                                                                                                                                        \
         kernel<<<grid, kGWarps * 32, smem, st>>>((const bf16 *)q, q_token, q_head, (const bf16 *)slab, num_pages, page_size, kv_heads * (dk + dv), dk, dv, \
                                                  heads, kv_heads, hp, block_table, max_pages, tiles, tok_pos, mask, mask_size, keep_first, scale, softcap, sink, \
-                                                 (const bf16 *)gate, g_token, (bf16 *)out, o_token, o_head, k_stride, v_stride, part, head_bias, weights); \
+                                                 (const bf16 *)gate, g_token, gate_wide, (bf16 *)out, o_token, o_head, k_stride, v_stride, part, head_bias, weights); \
     } while (0)
     if (pairs == 1) TLB_PAM(1);
     else if (pairs == 2) TLB_PAM(2);
@@ -410,7 +413,7 @@ int tlb_paged_attention_mma(const void *q, long long q_token, long long q_head, 
     TL_LAUNCH_CHECK("paged_attention_mma");
     if (splits > 1) {
         paged_attention_merge_kernel<<<dim3(num_tiles, kv_heads * ceil_div(group, hp), kGRows), 128, 0, st>>>(
-            part, splits, 64 * pairs + 2, tiles, heads, kv_heads, hp, dv, (const bf16 *)gate, g_token, (bf16 *)out, o_token, o_head);
+            part, splits, 64 * pairs + 2, tiles, heads, kv_heads, hp, dv, (const bf16 *)gate, g_token, gate_wide, (bf16 *)out, o_token, o_head);
         TL_LAUNCH_CHECK("paged_attention_merge");
     }
     return TL_OK;

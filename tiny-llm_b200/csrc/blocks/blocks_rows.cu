@@ -45,18 +45,6 @@ __global__ void embed_rows_kernel(const int32_t *__restrict__ ids, const T *__re
     }
 }
 
-// 4 consecutive elements of a row as floats (one 8- or 16-byte access)
-__device__ __forceinline__ float4 load4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
-__device__ __forceinline__ float4 load4(const bf16 *p) {
-    uint2 u = *reinterpret_cast<const uint2 *>(p);
-    float2 a = tl::unpack2<bf16>(u.x), b = tl::unpack2<bf16>(u.y);
-    return make_float4(a.x, a.y, b.x, b.y);
-}
-__device__ __forceinline__ void store4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
-__device__ __forceinline__ void store4(bf16 *p, float4 v) {
-    *reinterpret_cast<uint2 *>(p) = make_uint2(tl::pack2<bf16>(v.x, v.y), tl::pack2<bf16>(v.z, v.w));
-}
-
 // VEC: rows are read and written 4 elements at a time (dim % 4 == 0, 16-byte aligned bases); the row's values stay in
 // registers between the two passes when it has at most 4 * KEEP * blockDim elements.
 template <typename T, typename TY, bool VEC>
@@ -314,12 +302,6 @@ __global__ void latent_append_kernel(const T *__restrict__ down, const T *__rest
     for (int d = rot_dims + threadIdx.x; d < rot; d += blockDim.x) dst[rank + d] = src[rank + d];  // entries past the rotated ones pass
 }
 
-__device__ __forceinline__ float act_apply(float z, int act) {
-    if (act == 0) return z / (1.0f + expf(-z));
-    float inner = 0.7978845608028654f * (z + 0.044715f * z * z * z);
-    return 0.5f * z * (1.0f + tanhf(inner));
-}
-
 // out = act(x) elementwise; act 0 = silu, 1 = gelu (tanh form), 2 = squared relu, 4 = tanh.
 template <typename T>
 __global__ void act_rows_kernel(const T *__restrict__ x, T *__restrict__ out, long long total, int act) {
@@ -341,14 +323,6 @@ __global__ void cast_rows_kernel(const float *__restrict__ src, T *__restrict__ 
     const float *s = src + (size_t)blockIdx.x * dim;
     T *d = dst + (size_t)blockIdx.x * dst_stride;
     for (int i = threadIdx.x; i < dim; i += blockDim.x) d[i] = from_f<T>(s[i]);
-}
-
-__device__ __forceinline__ float gated_pair(float g, float u, int act, float limit, float slope) {
-    if (act == 3) {  // clamped: the gate from above, the other half on both sides; g sigmoid(slope g) (u + 1)
-        g = fminf(g, limit), u = fminf(fmaxf(u, -limit), limit);
-        return g / (1.0f + expf(-slope * g)) * (u + 1.0f);
-    }
-    return act_apply(g, act) * u;
 }
 
 template <typename T>
@@ -416,7 +390,7 @@ using namespace tlb;
 
 extern "C" {
 
-int tlb_abi_version(void) { return 6; }
+int tlb_abi_version(void) { return 7; }
 const char *tlb_last_error(void) { return tl::g_error; }
 long long tlb_launch_count(void) { return tl::g_launches.load(std::memory_order_relaxed); }
 

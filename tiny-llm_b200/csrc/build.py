@@ -52,6 +52,8 @@ BLOCKS_SOURCES = [
     "blocks/blocks_linear_attention.cu",
     "blocks/blocks_delta_rule.cu",
     "blocks/blocks_streams.cu",
+    "blocks/blocks_tanh_norm.cu",
+    "blocks/blocks_matrix_memory.cu",
 ]
 
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")

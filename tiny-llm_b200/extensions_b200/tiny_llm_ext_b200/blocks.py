@@ -40,28 +40,28 @@ _SIGNATURES = {
     "tlb_gated_act": (_I, [_VP, _VP, _LL, _I, _I, _I, _F, _F, _I, _VP]),
     "tlb_streams_step": (_I, [_VP, _VP, _VP, _VP, _VP, _VP, _F, _VP, _I, _I, _I, _I, _VP]),
     "tlb_shift_mix": (_I, [_VP, _LL, _VP, _I, _I, _VP, _I, _I, _VP, _LL, _I, _VP, _LL, _I, _VP]),
-    "tlb_moe_route": (_I, [_VP, _VP, _VP, _I, _I, _I, _I, _I, _VP, _F, _VP, _VP, _I, _VP]),
+    "tlb_moe_route": (_I, [_VP, _VP, _VP, _I, _I, _I, _I, _I, _VP, _F, _I, _I, _VP, _VP, _VP, _VP, _I, _VP]),
     "tlb_moe_up": (_I, [_VP, _VP, _VP, _VP, _VP, _I, _I, _I, _I, _I, _I, _I, _I, _VP, _I, _VP]),
     "tlb_moe_scale_rows": (_I, [_VP, _VP, _VP, _I, _I, _I, _I, _VP]),
     "tlb_add_norm": (_I, [_VP, _VP, _I, _VP, _VP, _F, _VP, _VP, _VP, _I, _I, _I, _VP]),
     "tlb_norm_mix2": (_I, [_VP, _VP, _VP, _VP, _F, _F, _VP, _I, _I, _I, _VP]),
     "tlb_paged_attention_tile_tokens": (_I, [_I, _I]),
-    "tlb_paged_attention": (_I, [_VP, _LL, _LL, _VP, _I, _I, _I, _I, _I, _I, _VP, _I, _VP, _I, _VP, _I, _I, _I, _F, _F, _I, _VP, _LL, _VP, _LL, _LL, _VP, _I, _I,
+    "tlb_paged_attention": (_I, [_VP, _LL, _LL, _VP, _I, _I, _I, _I, _I, _I, _VP, _I, _VP, _I, _VP, _I, _I, _I, _F, _F, _I, _VP, _LL, _I, _VP, _LL, _LL, _VP, _I, _I,
                                  _VP]),
     "tlb_paged_attention_mma_tile_tokens": (_I, [_I, _I]),
     "tlb_paged_attention_mma_supported": (_I, [_I, _I, _I, _I]),
-    "tlb_paged_attention_mma": (_I, [_VP, _LL, _LL, _VP, _I, _I, _I, _I, _I, _I, _VP, _I, _VP, _I, _VP, _I, _I, _I, _F, _F, _I, _VP, _LL, _VP, _LL, _LL, _I, _VP,
+    "tlb_paged_attention_mma": (_I, [_VP, _LL, _LL, _VP, _I, _I, _I, _I, _I, _I, _VP, _I, _VP, _I, _VP, _I, _I, _I, _F, _F, _I, _VP, _LL, _I, _VP, _LL, _LL, _I, _VP,
                                      ctypes.c_size_t, _VP, _I, _VP]),
     "tlb_paged_attention_mma_workspace": (ctypes.c_size_t, [_I, _I, _I, _I, _I]),
     "tlb_paged_attention_flash_tile_tokens": (_I, [_I, _I, _I]),
     "tlb_paged_attention_flash_supported": (_I, [_I, _I, _I, _I]),
-    "tlb_paged_attention_flash": (_I, [_VP, _LL, _LL, _VP, _I, _I, _I, _I, _I, _I, _VP, _I, _VP, _I, _VP, _I, _I, _I, _F, _F, _I, _VP, _LL, _VP, _LL, _LL, _I, _I,
+    "tlb_paged_attention_flash": (_I, [_VP, _LL, _LL, _VP, _I, _I, _I, _I, _I, _I, _VP, _I, _VP, _I, _VP, _I, _I, _I, _F, _F, _I, _VP, _LL, _I, _VP, _LL, _LL, _I, _I,
                                        _VP, _I, _VP]),
     "tlb_kv_prepare": (_I, [_VP, _LL, _LL, _I, _VP, _VP, _LL, _LL, _VP, _LL, _LL, _I, _I, _I, _VP, _F, _VP, _VP, _VP, _I, _I, _I, _VP, _I, _I, _VP]),
     "tlb_qk_whole_prepare": (_I, [_VP, _LL, _I, _VP, _VP, _LL, _VP, _LL, _I, _I, _I, _VP, _F, _I, _I, _D, _VP, _VP, _VP, _I, _I, _I, _VP, _VP, _VP, _I, _I, _VP]),
     "tlb_decay_scan_workspace": (ctypes.c_size_t, [_I, _I, _I, _I, _I]),
     "tlb_decay_scan": (_I, [_VP, _LL, _LL, _VP, _LL, _LL, _VP, _LL, _LL, _VP, _LL, _VP, _F, _VP, _VP, _VP, _I, _I, _F, _I, _I, _I, _VP, _I, _I, _VP, _LL, _I,
-                            _VP, _VP, ctypes.c_size_t, _I, _VP, _VP, _I, _VP, _I, _VP]),
+                            _VP, _VP, ctypes.c_size_t, _I, _VP, _VP, _I, _VP, _I, _I, _VP]),
     "tlb_delta_scan_workspace": (ctypes.c_size_t, [_I, _I, _I, _I, _I]),
     "tlb_delta_scan": (_I, [_VP, _LL, _LL, _VP, _LL, _LL, _VP, _LL, _LL, _VP, _LL, _VP, _I, _LL, _I, _VP, _VP, _F, _F, _I, _I, _I, _I, _VP, _I, _I, _VP, _LL,
                             _I, _VP, _VP, ctypes.c_size_t, _I, _VP]),
@@ -69,22 +69,27 @@ _SIGNATURES = {
     "tlb_act_rows": (_I, [_VP, _VP, _I, _I, _I, _I, _VP]),
     "tlb_softcap_rows": (_I, [_VP, _I, _I, _F, _VP]),
     "tlb_cast_rows": (_I, [_VP, _VP, _LL, _I, _I, _I, _VP]),
-    "tlb_head_norm_gate": (_I, [_VP, _VP, _F, _VP, _LL, _I, _VP, _I, _I, _I, _I, _I, _I, _VP]),
+    "tlb_head_norm_gate": (_I, [_VP, _VP, _F, _VP, _LL, _I, _VP, _I, _I, _I, _I, _I, _I, _VP, _F, _I, _VP]),
+    "tlb_matrix_memory_gates": (_I, [_VP, _LL, _VP, _LL, _VP, _I, _VP, _F, _I, _VP, _I, _I, _VP, _LL, _I, _VP, _VP, _I, _VP]),
+    "tlb_tanh_embed": (_I, [_VP, _VP, _I, _VP, _F, _VP, _VP, _F, _VP, _VP, _VP, _I, _I, _I, _VP]),
+    "tlb_tanh_step": (_I, [_VP, _VP, _VP, _F, _VP, _VP, _F, _VP, _VP, _VP, _I, _I, _I, _VP]),
+    "tlb_tanh_rows": (_I, [_VP, _VP, _F, _VP, _VP, _VP, _I, _I, _I, _VP]),
+    "tlb_moe_combine_tanh": (_I, [_VP, _VP, _VP, _VP, _VP, _VP, _I, _VP, _I, _F, _VP, _VP, _F, _VP, _VP, _VP, _I, _I, _I, _VP]),
     "tlb_moe_max_rows": (_LL, [_I, _I, _I, _I]),
     "tlb_moe_sort": (_I, [_VP, _I, _I, _I, _I, _VP, _VP, _VP, _VP]),
-    "tlb_moe_gate_up": (_I, [_VP, _VP, _VP, _VP, _VP, _VP, _I, _I, _I, _I, _I, _I, _I, _VP, _I, _VP]),
+    "tlb_moe_gate_up": (_I, [_VP, _VP, _VP, _VP, _VP, _VP, _I, _I, _I, _I, _I, _I, _I, _F, _F, _VP, _I, _VP]),
     "tlb_moe_down": (_I, [_VP, _VP, _VP, _VP, _VP, _I, _I, _I, _I, _I, _I, _VP, _I, _VP]),
-    "tlb_moe_combine": (_I, [_VP, _VP, _VP, _VP, _I, _VP, _VP, _I, _I, _I, _I, _VP]),
+    "tlb_moe_combine": (_I, [_VP, _VP, _VP, _VP, _VP, _I, _VP, _VP, _I, _I, _I, _I, _VP]),
     "tlb_argmax_rows": (_I, [_VP, _VP, _I, _I, _VP]),
 }
 EXPORTED_SYMBOLS = tuple(_SIGNATURES)
 
-ABI_VERSION = 6
+ABI_VERSION = 7
 ATTENTION_TILE_TOKENS = 4
 MOE_TILE_ROWS = 32
 ACT_SILU, ACT_GELU_TANH, ACT_RELU_SQUARED, ACT_CLAMPED_SWISH, ACT_TANH = 0, 1, 2, 3, 4
 WEIGHTS_SOFTMAX, WEIGHTS_SIGMOID = 0, 1
-DECAY_SIGMOID, DECAY_DOUBLE_EXP, DECAY_STEP = 0, 2, 3
+DECAY_SIGMOID, DECAY_DOUBLE_EXP, DECAY_STEP, DECAY_GIVEN = 0, 2, 3, 4
 MASK_CAUSAL, MASK_WINDOW, MASK_CHUNK = 0, 1, 2
 SCORE_SOFTMAX, SCORE_SIGMOID, SCORE_SOFTMAX_ALL = 0, 1, 2
 _DTYPE_CODE = {torch.float32: 0, torch.bfloat16: 2}
@@ -395,30 +400,41 @@ def gated_act(gate_up: torch.Tensor, act: int, limit: float = 0.0, slope: float 
     return out
 
 
-def moe_route(h, router_w, router_b, top: int, scoring: int = SCORE_SOFTMAX, choice_bias=None, weight_scale: float = 1.0):
+def moe_route(h, router_w, router_b, top: int, scoring: int = SCORE_SOFTMAX, choice_bias=None, weight_scale: float = 1.0, groups=(0, 0), side_w=None):
     """-> (expert ids int32 [T, top], weights fp32 [T, top]): softmax over the chosen logits, each one's sigmoid, or
     (``SCORE_SOFTMAX_ALL``) a softmax over all outputs, chosen by score + ``choice_bias``, the chosen scores renormalised
-    and times ``weight_scale``."""
-    _gpu("moe_route", h, router_w, router_b, choice_bias)
-    _contig("moe_route", h, router_w, router_b, choice_bias)
+    and times ``weight_scale``.  ``groups`` = (count, keep): the outputs form ``count`` equal runs of neighbours and only those of
+    the ``keep`` runs with the largest best choice score may be chosen.  ``side_w [1, D]``: a third result, fp32 ``[T]`` =
+    ``sigmoid(side_w . h)``."""
+    _gpu("moe_route", h, router_w, router_b, choice_bias, side_w)
+    _contig("moe_route", h, router_w, router_b, choice_bias, side_w)
+    if side_w is not None and (side_w.dtype != h.dtype or side_w.numel() != h.shape[1]):
+        raise RuntimeError("moe_route: side_w must be [1, D] of the activations' dtype")
     if choice_bias is not None and (choice_bias.dtype != h.dtype or choice_bias.numel() != router_w.shape[0]):
         raise RuntimeError("moe_route: choice_bias must be [experts] of the activations' dtype")
     T, D = h.shape
     E = router_w.shape[0]
     idx = torch.empty((T, top), dtype=torch.int32, device=h.device)
     gate = torch.empty((T, top), dtype=torch.float32, device=h.device)
-    _check(library().tlb_moe_route(_ptr(h), _ptr(router_w), _ptr(router_b), T, D, E, top, int(scoring), _ptr(choice_bias), float(weight_scale), _ptr(idx),
-                                   _ptr(gate), _code(h.dtype), _stream(h)))
-    return idx, gate
+    side = None if side_w is None else torch.empty(T, dtype=torch.float32, device=h.device)
+    _check(library().tlb_moe_route(_ptr(h), _ptr(router_w), _ptr(router_b), T, D, E, top, int(scoring), _ptr(choice_bias), float(weight_scale), int(groups[0]),
+                                   int(groups[1]), _ptr(side_w), _ptr(side), _ptr(idx), _ptr(gate), _code(h.dtype), _stream(h)))
+    return (idx, gate) if side_w is None else (idx, gate, side)
 
 
-def moe_experts(h, idx, gate, w_gate, w_up, w_down, act: int, shared=None, scale_input: bool = False, identity: bool = False) -> torch.Tensor:
+def moe_experts(h, idx, gate, w_gate, w_up, w_down, act: int, shared=None, scale_input: bool = False, identity: bool = False, limit: float = 0.0,
+                slope: float = 1.0, shared_gate=None, into=None, before_sum=None):
     """Sum of the chosen experts' feed-forwards (+ ``shared [T, D]``) -> fp32 ``[T, D]``.  ``w_up [E, ff, D]``,
     ``w_down [E, D, ff]``; with ``w_gate [E, ff, D]`` an expert is ``down(act(gate x) * (up x))``, without it
     ``down(act(up x))``.  The router's weight multiplies the expert's output, or, ``scale_input``, its input ``x``
-    (rounded to the compute dtype).  ``identity``: ids from ``E`` up name identity experts, whose output is the token itself."""
-    _gpu("moe_experts", h, idx, gate, w_gate, w_up, w_down, shared)
-    _contig("moe_experts", h, idx, gate, w_gate, w_up, w_down, shared)
+    (rounded to the compute dtype).  ``identity``: ids from ``E`` up name identity experts, whose output is the token itself.
+    ``limit`` and ``slope`` go with ``ACT_CLAMPED_SWISH`` (see ``gated_act``); ``shared_gate`` (fp32 ``[T]``) multiplies ``shared``.
+    ``into`` = (stream fp32 ``[T, D]``, post norm, next norm or None): instead of being returned, the sum passes the post norm into
+    the stream (in place), and the next norm of the new stream is returned (``tanh_step``).  ``before_sum()`` is called ahead of the launch that reads ``shared``."""
+    _gpu("moe_experts", h, idx, gate, w_gate, w_up, w_down, shared, shared_gate)
+    _contig("moe_experts", h, idx, gate, w_gate, w_up, w_down, shared, shared_gate)
+    if shared_gate is not None and (shared_gate.dtype != torch.float32 or shared_gate.shape != (h.shape[0],)):
+        raise RuntimeError("moe_experts: shared_gate must be float32 [T]")
     lib = library()
     T, D = h.shape
     E, ff, _ = w_up.shape
@@ -432,7 +448,6 @@ def moe_experts(h, idx, gate, w_gate, w_up, w_down, act: int, shared=None, scale
     counters = torch.empty(2, dtype=torch.int32, device=dev)
     inter = torch.empty((max_rows, ff), dtype=h.dtype, device=dev)
     pair_out = torch.empty((T * top, D), dtype=torch.float32, device=dev)
-    y = torch.empty((T, D), dtype=torch.float32, device=dev)
     _check(lib.tlb_moe_sort(_ptr(idx), T, top, E, rows, _ptr(sorted_pair), _ptr(tile_expert), _ptr(counters), st))
     rows_in, per_pair = h, 0
     if scale_input:
@@ -442,14 +457,83 @@ def moe_experts(h, idx, gate, w_gate, w_up, w_down, act: int, shared=None, scale
         if per_pair:
             raise RuntimeError("moe_experts: gated experts take the router's weight on their output")
         _check(lib.tlb_moe_gate_up(_ptr(h), _ptr(w_gate), _ptr(w_up), _ptr(sorted_pair), _ptr(tile_expert), _ptr(counters), T, top, E, rows, D, ff, act,
-                                   _ptr(inter), code, st))
+                                   float(limit), float(slope), _ptr(inter), code, st))
     else:
         _check(lib.tlb_moe_up(_ptr(rows_in), _ptr(w_up), _ptr(sorted_pair), _ptr(tile_expert), _ptr(counters), T, top, E, rows, D, ff, act, per_pair,
                               _ptr(inter), code, st))
     _check(lib.tlb_moe_down(_ptr(inter), _ptr(w_down), _ptr(sorted_pair), _ptr(tile_expert), _ptr(counters), T, top, E, rows, D, ff, _ptr(pair_out), code, st))
-    _check(lib.tlb_moe_combine(_ptr(pair_out), None if scale_input else _ptr(gate), _ptr(shared), _ptr(idx) if identity else None, E,
+    if before_sum is not None:
+        before_sum()
+    if into is not None:
+        x, post, following = into
+        if scale_input:
+            raise RuntimeError("moe_experts: a fused step takes the router's weight on the experts' output")
+        out = _tanh_out("moe_experts", x, post, following)
+        if post.weight.dtype != h.dtype or x.shape != (T, D):
+            raise RuntimeError("moe_experts: stream [T, D] and norms of the activations' dtype")
+        _check(lib.tlb_moe_combine_tanh(_ptr(x), _ptr(pair_out), _ptr(gate), _ptr(shared), _ptr(shared_gate), _ptr(idx) if identity else None, E,
+                                        _ptr(h) if identity else None, top, *_tanh_args(post), *_tanh_args(following), _ptr(out), T, D, code, st))
+        return out
+    y = torch.empty((T, D), dtype=torch.float32, device=dev)
+    _check(lib.tlb_moe_combine(_ptr(pair_out), None if scale_input else _ptr(gate), _ptr(shared), _ptr(shared_gate), _ptr(idx) if identity else None, E,
                                _ptr(h) if identity else None, _ptr(y), T, top, D, code, st))
     return y
+
+
+def _tanh_args(norm) -> tuple:
+    return (0.0, None, None) if norm is None else (norm.alpha, _ptr(norm.weight), _ptr(norm.bias))
+
+
+def _tanh_out(op: str, x, post, following, rows: int | None = None):
+    """Checks one step's norms (objects with ``weight``, ``bias`` and the number ``alpha``) -> the next norm's output, or None."""
+    _gpu(op, x)
+    _contig(op, x)
+    if x.dtype != torch.float32 or x.dim() != 2:
+        raise RuntimeError(f"{op}: the stream must be float32 [rows, dim]")
+    for n in (post, following):
+        if n is not None and (n.weight.shape != x.shape[1:] or n.bias.shape != x.shape[1:] or n.weight.dtype != n.bias.dtype or not n.weight.is_contiguous() or not n.bias.is_contiguous()):
+            raise RuntimeError(f"{op}: a norm's weight and bias must be [dim] of one dtype")
+    if post is not None and following is not None and post.weight.dtype != following.weight.dtype:
+        raise RuntimeError(f"{op}: norms of one dtype")
+    return None if following is None else torch.empty((x.shape[0] if rows is None else rows, x.shape[1]), dtype=following.weight.dtype, device=x.device)
+
+
+def tanh_embed(ids, table, post, following):
+    """The start of a stream behind an elementwise norm: ``x = post(table[ids])`` fp32 -> (x, ``following(x)`` in the norms' dtype);
+    a norm is ``weight * tanh(alpha * x) + bias``."""
+    _gpu("tanh_embed", ids, table)
+    _contig("tanh_embed", ids, table)
+    if ids.dtype != torch.int32 or ids.dim() != 1 or table.dim() != 2 or table.dtype != post.weight.dtype:
+        raise RuntimeError("tanh_embed: int32 ids [T] and a table [vocab, dim] of the norms' dtype")
+    x = torch.empty((ids.numel(), table.shape[1]), dtype=torch.float32, device=table.device)
+    h = _tanh_out("tanh_embed", x, post, following)
+    _check(library().tlb_tanh_embed(_ptr(ids), _ptr(table), table.shape[0], _ptr(x), *_tanh_args(post), *_tanh_args(following), _ptr(h), x.shape[0], x.shape[1],
+                                    _code(table.dtype), _stream(table)))
+    return x, h
+
+
+def tanh_step(x, y, post, following, y_bias=None):
+    """``x += post(y + y_bias)`` (fp32 ``[rows, dim]``, in place), then ``following(x)`` rounded to the norms' dtype (None: not
+    wanted); norms as for ``tanh_embed``."""
+    _gpu("tanh_step", x, y, y_bias)
+    _contig("tanh_step", y, y_bias)
+    if y.dtype != torch.float32 or y.shape != x.shape or (y_bias is not None and (y_bias.shape != x.shape[1:] or y_bias.dtype != post.weight.dtype)):
+        raise RuntimeError("tanh_step: y must be float32 of the stream's shape, y_bias [dim] of the norms' dtype")
+    h = _tanh_out("tanh_step", x, post, following)
+    _check(library().tlb_tanh_step(_ptr(x), _ptr(y), _ptr(y_bias), *_tanh_args(post), *_tanh_args(following), _ptr(h), x.shape[0], x.shape[1],
+                                   _code(post.weight.dtype), _stream(x)))
+    return h
+
+
+def tanh_rows(x, norm, rows=None):
+    """``norm`` of the stream's rows ``rows`` (int32; None = all), rounded to the norm's dtype."""
+    _gpu("tanh_rows", x, rows)
+    _contig("tanh_rows", rows)
+    if rows is not None and (rows.dtype != torch.int32 or rows.dim() != 1):
+        raise RuntimeError("tanh_rows: rows must be int32 [n]")
+    h = _tanh_out("tanh_rows", x, None, norm, None if rows is None else rows.numel())
+    _check(library().tlb_tanh_rows(_ptr(x), _ptr(rows), *_tanh_args(norm), _ptr(h), h.shape[0], x.shape[1], _code(h.dtype), _stream(x)))
+    return h
 
 
 def add_norm(residual: torch.Tensor, a: torch.Tensor, b: torch.Tensor | None, weight: torch.Tensor | None, eps: float, weight2: torch.Tensor | None = None):
@@ -586,7 +670,8 @@ def paged_attention(q, slab, block_table, tiles, tok_pos, *, kv_heads: int, dv: 
     the step, 0 = unknown) lets the tensor-core kernel split the key range over several CTAs when the launch alone would
     leave SMs idle.  ``head_bias`` (fp32 ``[H]``): with ``sink`` the sink's term is ``exp(head_bias[h])`` instead of ``exp(0)``;
     with ``weights=WEIGHTS_SIGMOID`` there is no softmax, a visible key weighs ``sigmoid(score + head_bias[h])``.  ``keep_first``
-    (window mask): the sequence's first positions that stay visible from everywhere after them."""
+    (window mask): the sequence's first positions that stay visible from everywhere after them.  A gate of ``[T, H * dv]`` has a
+    logit for every entry of every head."""
     _gpu("paged_attention", q, slab, block_table, tiles, tok_pos, gate, out, head_bias)
     if head_bias is not None and (head_bias.dtype != torch.float32 or head_bias.shape != (q.shape[1],) or not head_bias.is_contiguous()):
         raise RuntimeError("paged_attention: head_bias must be float32 [H]")
@@ -595,8 +680,9 @@ def paged_attention(q, slab, block_table, tiles, tok_pos, *, kv_heads: int, dv: 
     P, page_size, width = slab.shape
     if width != kv_heads * (dk + dv) or q.dtype != slab.dtype or q.stride(2) != 1:
         raise RuntimeError("paged_attention: query and cache do not match")
-    if gate is not None and (gate.shape != (T, H) or gate.stride(1) != 1 or gate.dtype != q.dtype):
-        raise RuntimeError("paged_attention: gate must be [T, H] of the query's dtype")
+    wide = int(gate is not None and gate.shape == (T, H * dv) and dv > 1)
+    if gate is not None and ((gate.shape != (T, H) and not wide) or gate.stride(1) != 1 or gate.dtype != q.dtype):
+        raise RuntimeError("paged_attention: gate must be [T, H] or [T, H * dv] of the query's dtype")
     if out is None:
         out = torch.empty((T, H, dv), dtype=q.dtype, device=q.device)
     elif out.shape != (T, H, dv) or out.dtype != q.dtype or out.stride(2) != 1:
@@ -609,7 +695,7 @@ def paged_attention(q, slab, block_table, tiles, tok_pos, *, kv_heads: int, dv: 
         splits = flash_splits(tiles.shape[0] * kv_heads * -(-group // rows), max_context, most, slab.device) if max_context else 1
         _check(library().tlb_paged_attention_flash(_ptr(q), q.stride(0), q.stride(1), _ptr(slab), P, page_size, dk, dv, H, kv_heads, _ptr(block_table),
                                                    block_table.shape[1], _ptr(tiles), tiles.shape[0], _ptr(tok_pos), int(mask), int(mask_size), int(keep_first),
-                                                   float(scale), float(softcap or 0.0), int(bool(sink)), _ptr(gate), gate.stride(0) if gate is not None else 0,
+                                                   float(scale), float(softcap or 0.0), int(bool(sink)), _ptr(gate), gate.stride(0) if gate is not None else 0, wide,
                                                    _ptr(out), out.stride(0), out.stride(1), int(kernel == "flash_split"), splits, _ptr(head_bias), int(weights),
                                                    _stream(q)))
         return out
@@ -626,20 +712,20 @@ def paged_attention(q, slab, block_table, tiles, tok_pos, *, kv_heads: int, dv: 
         _check(lib.tlb_paged_attention_mma(_ptr(q), q.stride(0), q.stride(1), _ptr(slab), P, page_size, dk, dv, H, kv_heads, _ptr(block_table),
                                            block_table.shape[1], _ptr(tiles), tiles.shape[0], _ptr(tok_pos), int(mask), int(mask_size), int(keep_first),
                                            float(scale), float(softcap or 0.0), int(bool(sink)), _ptr(gate),
-                                           gate.stride(0) if gate is not None else 0, _ptr(out), out.stride(0), out.stride(1), splits, _ptr(ws), nbytes,
+                                           gate.stride(0) if gate is not None else 0, wide, _ptr(out), out.stride(0), out.stride(1), splits, _ptr(ws), nbytes,
                                            _ptr(head_bias), int(weights), _stream(q)))
         return out
     if kernel != "general":
         raise RuntimeError(f"paged_attention: unknown kernel {kernel!r}")
     _check(library().tlb_paged_attention(_ptr(q), q.stride(0), q.stride(1), _ptr(slab), P, page_size, dk, dv, H, kv_heads, _ptr(block_table),
                                          block_table.shape[1], _ptr(tiles), tiles.shape[0], _ptr(tok_pos), int(mask), int(mask_size), int(keep_first), float(scale),
-                                         float(softcap or 0.0), int(bool(sink)), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(out),
+                                         float(softcap or 0.0), int(bool(sink)), _ptr(gate), gate.stride(0) if gate is not None else 0, wide, _ptr(out),
                                          out.stride(0), out.stride(1), _ptr(head_bias), int(weights), _code(q.dtype), _stream(q)))
     return out
 
 
 def decay_scan(q, k, v, z, z_bias, *, tau: float = 1.0, q_scale: float, seq_info, state, out=None, max_tokens: int | None = None, head_decay=None,
-               rope=None, rope_dims: int = 0, rope_interleaved: bool = False, decay_kind: int = 0, a_log=None, bonus=None, skip=None):
+               rope=None, rope_dims: int = 0, rope_interleaved: bool = False, decay_kind: int = 0, a_log=None, bonus=None, skip=None, normaliser: bool = False):
     """Linear attention with per-channel decay ``sigmoid(z + z_bias)^(1/tau)``: ``q, k [T, H, dk]``, ``v [T, H, dv]`` views,
     ``z [T, H * dk]`` fp32, ``seq_info [S, 4]`` int32 (first token, count, start position, slot), ``state [slots, H, dk, dv]``
     fp32 (a view whose slots may be further apart) -> fp32 ``[T, H, dv]``.  ``max_tokens``: the largest count in
@@ -650,18 +736,23 @@ def decay_scan(q, k, v, z, z_bias, *, tau: float = 1.0, q_scale: float, seq_info
     ``DECAY_STEP`` = one decay per head and token, ``exp(-exp(a_log[h]) dt)`` with ``dt = softplus(z[t, h] + z_bias[h])``
     (``z [T, H]``), the key multiplied by ``dt``.  ``q, k`` may have fewer heads than ``v`` (``[T, G, dk]``, head h reads
     ``h // (H // G)``).  ``skip [H]``: ``out += skip[h] v``.  ``bonus [H, dk]``: the read-out comes before the update and
-    weighs the token's own ``k v^T`` by it."""
+    weighs the token's own ``k v^T`` by it.  ``DECAY_GIVEN``: ``z [T, H, 2]`` holds one (decay, key factor) pair per head and token.
+    ``normaliser``: the state and the output have one more column, ``[.., dv + 1]``, in which every value is 1."""
     _gpu("decay_scan", q, k, v, z, z_bias, seq_info, state, out, head_decay, a_log, bonus, skip)
     T, G, dk = q.shape
     H, dv = v.shape[1], v.shape[2]
     if k.shape != (T, G, dk) or v.shape[0] != T or H % G:
         raise RuntimeError("decay_scan: shapes do not match")
+    v_cols, dv = dv, dv + int(normaliser)
     for name, t, shape in (("a_log", a_log, (H,)), ("bonus", bonus, (H, dk)), ("skip", skip, (H,))):
         if t is not None and (t.shape != shape or t.dtype != q.dtype or not t.is_contiguous()):
             raise RuntimeError(f"decay_scan: {name} must be {shape} of the activations' dtype")
     if decay_kind == DECAY_STEP:
         if z is None or z.shape != (T, H) or z.dtype != torch.float32 or z.stride(1) != 1 or a_log is None or head_decay is not None:
             raise RuntimeError("decay_scan: a step decay takes z [T, H] float32 and a_log [H]")
+    elif decay_kind == DECAY_GIVEN:
+        if z is None or z.shape != (T, H, 2) or z.dtype != torch.float32 or not z.is_contiguous() or z_bias is not None or head_decay is not None:
+            raise RuntimeError("decay_scan: given decays are float32 [T, H, 2]")
     elif head_decay is not None:
         if z is not None or head_decay.dtype != torch.float32 or head_decay.shape != (H,) or not head_decay.is_contiguous():
             raise RuntimeError("decay_scan: head_decay must be float32 [H] and replaces z")
@@ -689,19 +780,23 @@ def decay_scan(q, k, v, z, z_bias, *, tau: float = 1.0, q_scale: float, seq_info
     _check(lib.tlb_decay_scan(_ptr(q), q.stride(0), q.stride(1), _ptr(k), k.stride(0), k.stride(1), _ptr(v), v.stride(0), v.stride(1), _ptr(z),
                               z.stride(0) if z is not None else 0, _ptr(z_bias), float(tau), _ptr(head_decay), _ptr(cs), _ptr(sn), int(rope_dims),
                               int(bool(rope_interleaved)), float(q_scale), H, dk, dv, _ptr(seq_info), seq_info.shape[0], longest, _ptr(state),
-                              state.stride(0), state.shape[0], _ptr(out), _ptr(ws), nbytes, int(decay_kind), _ptr(a_log), _ptr(bonus), G, _ptr(skip),
+                              state.stride(0), state.shape[0], _ptr(out), _ptr(ws), nbytes, int(decay_kind), _ptr(a_log), _ptr(bonus), G, _ptr(skip), v_cols,
                               _code(q.dtype), _stream(q)))
     return out
 
 
-def head_norm_gate(o, weight, eps: float, gate=None, act: int = 1, gate_first: bool = False):
+def head_norm_gate(o, weight, eps: float, gate=None, act: int = 1, gate_first: bool = False, floor=None, den_eps: float = 0.0):
     """``o [T, H, dv]`` fp32 -> ``[T, H * dv]`` in the weight's (without one: the gate's) dtype: per-head RMS norm times
     ``weight [dv]`` (None = no weight) times ``silu(gate)`` (``act`` 1), ``sigmoid(gate)`` (2) or ``gate`` (0);
     ``gate [T, H * dv]`` a view with unit inner stride.  A weight of ``[H * dv]`` gives every head its own part;
-    ``gate_first``: the gate multiplies ``o`` BEFORE the norm."""
-    _gpu("head_norm_gate", o, weight, gate)
-    _contig("head_norm_gate", o, weight)
-    T, H, dv = o.shape
+    ``gate_first``: the gate multiplies ``o`` BEFORE the norm.  ``floor`` (fp32 ``[T, H]``): ``o [T, H, dv + 1]`` ends in a normaliser
+    and is first divided by ``max(|o[.., dv]|, floor) + den_eps``."""
+    _gpu("head_norm_gate", o, weight, gate, floor)
+    _contig("head_norm_gate", o, weight, floor)
+    T, H, row = o.shape
+    dv = row - int(floor is not None)
+    if floor is not None and (floor.dtype != torch.float32 or floor.shape != (T, H)):
+        raise RuntimeError("head_norm_gate: floor must be float32 [T, H]")
     if weight is None and gate is None:
         raise RuntimeError("head_norm_gate: a weight or a gate must name the output dtype")
     dtype = weight.dtype if weight is not None else gate.dtype
@@ -710,8 +805,33 @@ def head_norm_gate(o, weight, eps: float, gate=None, act: int = 1, gate_first: b
         raise RuntimeError("head_norm_gate: shapes do not match")
     out = torch.empty((T, H * dv), dtype=dtype, device=o.device)
     _check(library().tlb_head_norm_gate(_ptr(o), _ptr(weight), float(eps), _ptr(gate), gate.stride(0) if gate is not None else 0, int(act), _ptr(out),
-                                        T, H, dv, int(wide), int(bool(gate_first)), _code(dtype), _stream(o)))
+                                        T, H, dv, int(wide), int(bool(gate_first)), row, _ptr(floor), float(den_eps), _code(dtype), _stream(o)))
     return out
+
+
+def matrix_memory_gates(z, *, h=None, w=None, bias, cap: float, heads: int, seq_info, state, max_tokens: int):
+    """Log gates of a matrix memory to the numbers of its recurrence: ``z [T, 2 * heads]`` fp32 (input gates, forget gates), or None
+    and the products of ``h [T, D]`` with ``w [2 * heads, D]`` made by the kernel; ``bias [2 * heads]``; ``state [slots, heads]`` fp32 (a
+    view), the running maximum -> (steps fp32 ``[T, heads, 2]`` for ``decay_scan`` with ``DECAY_GIVEN``, floor fp32 ``[T, heads]``)."""
+    _gpu("matrix_memory_gates", z, h, w, bias, seq_info, state)
+    _contig("matrix_memory_gates", w, bias, seq_info)
+    rows = z if z is not None else h
+    if z is not None and (z.dtype != torch.float32 or z.shape[1] != 2 * heads or z.stride(1) != 1):
+        raise RuntimeError("matrix_memory_gates: z must be float32 [T, 2 * heads]")
+    if z is None and (w.shape != (2 * heads, h.shape[1]) or w.dtype != h.dtype or h.stride(1) != 1):
+        raise RuntimeError("matrix_memory_gates: w must be [2 * heads, D] of h's dtype")
+    if bias.numel() != 2 * heads or (z is None and bias.dtype != h.dtype):
+        raise RuntimeError("matrix_memory_gates: bias must be [2 * heads] of h's dtype")
+    if state.dtype != torch.float32 or state.shape[1:] != (heads,) or state.stride(1) != 1 or seq_info.dtype != torch.int32 or seq_info.shape[1:] != (4,):
+        raise RuntimeError("matrix_memory_gates: state must be float32 [slots, heads], seq_info int32 [S, 4]")
+    T = rows.shape[0]
+    step = torch.empty((T, heads, 2), dtype=torch.float32, device=rows.device)
+    floor = torch.empty((T, heads), dtype=torch.float32, device=rows.device)
+    _check(library().tlb_matrix_memory_gates(_ptr(z), z.stride(0) if z is not None else 0, _ptr(h) if z is None else None, h.stride(0) if z is None else 0,
+                                             _ptr(w) if z is None else None, w.shape[1] if z is None else 0, _ptr(bias), float(cap), int(heads), _ptr(seq_info),
+                                             seq_info.shape[0], max(1, int(max_tokens)), _ptr(state), state.stride(0), state.shape[0], _ptr(step), _ptr(floor),
+                                             _code(bias.dtype), _stream(rows)))
+    return step, floor
 
 
 def delta_scan(q, k, v, beta, a, a_log, dt_bias, *, per_channel: bool, q_scale: float, unit_eps: float = 1e-6, seq_info, state, out=None,

@@ -81,3 +81,30 @@ class ResidualStreams:
         from extensions_b200.tiny_llm_ext_b200 import blocks
 
         return blocks.streams_step(xs, y=y, y_bias=y_bias, write=write, read=read, eps=self.eps, dtype=self.dtype)
+
+
+class TanhNorm:
+    """The elementwise bounded norm ``weight * tanh(alpha * x) + bias`` (Dynamic Tanh): ``alpha`` one number, no statistics over the
+    row.  ``follow`` is one sublayer's end: its output passes this norm into the fp32 stream ``x`` (in place), and the norm
+    that reads the stream next is evaluated in the same launch; ``rows`` the norm alone, of some rows of the stream."""
+
+    def __init__(self, weight: torch.Tensor, bias: torch.Tensor, alpha: torch.Tensor):
+        if weight.dim() != 1 or bias.shape != weight.shape or alpha.numel() != 1:
+            raise ValueError("tanh norm: a weight and a bias of the width and one number alpha")
+        self.weight, self.bias, self.alpha = weight.contiguous(), bias.contiguous(), float(alpha)
+
+    def embed(self, ids: torch.Tensor, table: torch.Tensor, following: "TanhNorm"):
+        """-> (the stream ``self(table[ids])`` in fp32, ``following`` of it)."""
+        from extensions_b200.tiny_llm_ext_b200 import blocks
+
+        return blocks.tanh_embed(ids, table, self, following)
+
+    def follow(self, x: torch.Tensor, y: torch.Tensor, following: "TanhNorm | None", y_bias=None):
+        from extensions_b200.tiny_llm_ext_b200 import blocks
+
+        return blocks.tanh_step(x, y, self, following, y_bias)
+
+    def rows(self, x: torch.Tensor, rows=None) -> torch.Tensor:
+        from extensions_b200.tiny_llm_ext_b200 import blocks
+
+        return blocks.tanh_rows(x, self, rows)

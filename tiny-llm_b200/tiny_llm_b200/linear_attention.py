@@ -1,5 +1,6 @@
 """Linear attention with a decay: recurrent mixers whose state lives in fp32 slots.  ``DecayedLinearAttention`` has one
-input-dependent decay per key channel, ``RetainedLinearAttention`` (at the end of the file) one fixed decay per head.
+input-dependent decay per key channel, ``RetainedLinearAttention`` one fixed decay per head, ``ShiftedBonusLinearAttention`` token
+shift and a bonus for the current token, ``MatrixMemory`` exponential gates per head and a normaliser.
 
 Per head a matrix ``S [dim, vdim]`` is carried along the sequence,
 
@@ -131,3 +132,54 @@ class ShiftedBonusLinearAttention:
         o = blocks.decay_scan(rkvg[0].unflatten(1, (H, d)), rkvg[1].unflatten(1, (H, d)), rkvg[2].unflatten(1, (H, d)), z, self.w0, q_scale=1.0,
                               seq_info=plan.seq_info, state=state, max_tokens=plan.max_tokens, decay_kind=blocks.DECAY_DOUBLE_EXP, bonus=self.bonus)
         return linear_wide(blocks.head_norm_gate(o, self.norm_weight, self.eps, rkvg[3], act=1), self.w_o)
+
+
+class MatrixMemory:
+    """The matrix memory of xLSTM (mLSTM): an exponential input gate and a sigmoid forget gate per head, both from soft-capped
+    projections, and a read-out divided by a normaliser that is carried beside the memory,
+
+        i_t = cap tanh((W_i h + b_i) / cap)        f_t = log_sigmoid(cap tanh((W_f h + b_f) / cap))
+        m_t = max(f_t + m_(t-1), i_t)              (m_0 = 0)
+        S_t = e^(f_t + m_(t-1) - m_t) S_(t-1) + e^(i_t - m_t) k_t v_t^T        n_t likewise with k_t alone
+        o_t = S_t^T q_t / (max(|n_t . q_t|, e^(-m_t)) + 1e-6)                  (dim^-1/2 folded into q)
+
+    Each head's ``o`` is divided by its root mean square, multiplied by ``norm_weight`` (one entry per head and channel) and by
+    ``sigmoid(gate)``, and projected.  The running maximum is a scan of its own over two numbers per token and head
+    (``blocks.matrix_memory_gates``); with the decays it gives, memory and normaliser are one recurrence, the normaliser an extra
+    value column that is always 1 (``blocks.decay_scan``, so long portions run as parallel segments like those of the other
+    mixers); normaliser, norm and gate are one launch.  The gates' projections keep their fp32 accumulator, gates, recurrence and norm are
+    fp32 whatever the compute dtype.  A request's state is two blocks of its slot: ``state [slots, heads, dim, vdim + 1]`` and
+    the running maximum ``peak [slots, heads]``; both start from zero at position 0 whatever the slot held."""
+
+    DEN_EPS = 1e-6
+    INLINE_TOKENS = 2  # steps of at most this many tokens a sequence: the gates' launch makes its two small projections itself
+
+    def __init__(self, *, heads: int, dim: int, vdim: int, gate_cap: float, w_i, b_i, w_f, b_f, norm_weight, w_o, eps: float = 1e-6):
+        self.heads, self.dim, self.vdim, self.gate_cap, self.eps = int(heads), int(dim), int(vdim), float(gate_cap), float(eps)
+        if w_i.shape[0] != heads or w_f.shape != w_i.shape or b_i.numel() != heads or b_f.numel() != heads or not self.gate_cap > 0:
+            raise ValueError("matrix memory: one input and one forget gate per head, and a positive cap")
+        if norm_weight.numel() != heads * vdim or tuple(w_o.shape)[1] != heads * vdim:
+            raise ValueError("matrix memory: norm and output projection do not match heads x vdim")
+        self.w_gates, self.b_gates = torch.cat([w_i, w_f]).contiguous(), torch.cat([b_i.reshape(-1), b_f.reshape(-1)]).contiguous()
+        self.norm_weight, self.w_o = norm_weight.reshape(-1).contiguous(), w_o.contiguous()
+
+    @property
+    def state_shape(self) -> tuple:
+        return (self.heads, self.dim, self.vdim + 1)
+
+    @property
+    def peak_shape(self) -> tuple:
+        return (self.heads,)
+
+    def __call__(self, h, q, k, v, gate, plan, state: torch.Tensor, peak: torch.Tensor) -> torch.Tensor:
+        """``h [T, width]`` the mixer's input; ``q, k [T, heads * dim]``, ``v, gate [T, heads * vdim]`` views of the fused projection."""
+        from extensions_b200.tiny_llm_ext_b200 import blocks
+
+        H = self.heads
+        z = None if plan.max_tokens <= self.INLINE_TOKENS else linear_wide(h, self.w_gates)
+        steps, floor = blocks.matrix_memory_gates(z, h=h, w=self.w_gates, bias=self.b_gates, cap=self.gate_cap, heads=H, seq_info=plan.seq_info,
+                                                  state=peak, max_tokens=plan.max_tokens)
+        o = blocks.decay_scan(q.unflatten(1, (H, self.dim)), k.unflatten(1, (H, self.dim)), v.unflatten(1, (H, self.vdim)), steps, None,
+                              q_scale=self.dim ** -0.5, seq_info=plan.seq_info, state=state, max_tokens=plan.max_tokens,
+                              decay_kind=blocks.DECAY_GIVEN, normaliser=True)
+        return linear_wide(blocks.head_norm_gate(o, self.norm_weight, self.eps, gate, act=2, floor=floor, den_eps=self.DEN_EPS), self.w_o)

@@ -22,6 +22,7 @@ ARCHITECTURES = {
     "Senurax": ("tiny_llm_b200.senurax", "SenuraxModel"),
     "Norusun": ("tiny_llm_b200.norusun", "NorusunModel"),
     "Zalazen": ("tiny_llm_b200.zalazen", "ZalazenModel"),
+    "Nomudra": ("tiny_llm_b200.nomudra", "NomudraModel"),
 }
 
 

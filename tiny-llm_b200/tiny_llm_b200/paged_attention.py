@@ -2,18 +2,19 @@
 parameters: what a position sees (``mask`` = ``"causal"``, ``"window"``: itself and the ``mask_size - 1`` positions
 before it, plus the sequence's first ``keep_first`` positions at their true places, ``"chunk"``: the earlier positions of
 its own block of ``mask_size`` positions counted from 0), a tanh ``softcap`` on the scaled scores, a ``sink`` (one more term ``exp(0)`` in the softmax's denominator), per-head RMS
-norms of queries and keys (plain weights of size ``dim``, shared by the heads) and a sigmoid output gate per head
-(``gate`` None = no gate).  With ``rot`` = ``{"dims", "base", "factor", "interleaved"}`` the first ``dims`` entries of every
+norms of queries and keys (plain weights of size ``dim``, shared by the heads) and a sigmoid output gate per head or per entry of
+every head (``gate`` None = no gate).  With ``rot`` = ``{"dims", "base", "factor", "interleaved"}`` the first ``dims`` entries of every
 query and key head are rotated by the token's position (pairs ``(2i, 2i+1)`` or ``(i, i + dims/2)``, every frequency
 divided by ``factor``; with ``yarn`` = ``{"factor", "original", "fast", "slow"}`` stretched by frequency, ``positional_encoding.yarn_ramp``)
 before the keys are stored; without it the scores carry no positional term.
 ``qk_norm="whole"``: each norm takes a token's whole query (key) projection as one vector, ahead of the split into heads and
 before any rotation, with weights of that size.  ``head_bias`` (one learned number per head): with ``sink`` the sink's term is
 ``exp(head_bias[h])``; with ``weights="sigmoid"`` there is no softmax at all, a visible key weighs
-``sigmoid(score + head_bias[h])`` and nothing is normalised over the keys.
+``sigmoid(score + head_bias[h])`` and nothing is normalised over the keys.  ``values="keys"``: there is no value projection, the
+values are the keys as projected, ahead of the rotation (``v`` None).
 
 The layer's input projections are made by the caller in one product (``FusedProjection``); the module takes the views
-``q [T, H * dim]``, ``k [T, G * dim]``, ``v [T, G * vdim]`` and ``gate [T, H]`` (logits), stores keys and values in the
+``q [T, H * dim]``, ``k [T, G * dim]``, ``v [T, G * vdim]`` and ``gate [T, H]`` or ``[T, H * vdim]`` (logits), stores keys and values in the
 layer's slab ``[pages, page_size, G * (dim + vdim)]`` (or, built with ``caches=False``, reads another layer's slab and
 gets no k / v), runs the attention kernel over the plan's work list and returns the output projection in fp32.
 """
@@ -82,7 +83,7 @@ class JoinedProjection:
 class PagedGroupedAttention:
     def __init__(self, *, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, mask: str, mask_size: int, w_o, softcap: float | None = None,
                  sink: bool = False, q_norm=None, k_norm=None, eps: float = 1e-6, caches: bool = True, page_size: int = 64, rot: dict | None = None,
-                 qk_norm: str = "head", head_bias=None, weights: str = "softmax", keep_first: int = 0):
+                 qk_norm: str = "head", head_bias=None, weights: str = "softmax", keep_first: int = 0, values: str = "own"):
         if heads % kv_heads:
             raise ValueError(f"{heads} query heads do not divide into {kv_heads} key/value heads")
         if mask not in MASKS or (mask != "causal" and int(mask_size) <= 0):
@@ -108,6 +109,9 @@ class PagedGroupedAttention:
             raise ValueError("attention: one head_bias per head")
         if self.weights == WEIGHTS["sigmoid"] and (sink or softcap):
             raise ValueError("attention: sigmoid weights take no sink and no cap")
+        if values not in ("own", "keys") or (values == "keys" and (vdim != dim or not caches or (qk_norm == "head" and (q_norm is not None or k_norm is not None)))):
+            raise ValueError(f"attention: values={values!r} of {vdim} entries beside keys of {dim}")
+        self.tied_values = values == "keys"
         self.rot = None
         if rot and int(rot.get("dims", 0)) > 0:
             if (q_norm is not None or k_norm is not None) and not self.whole_norm:
@@ -155,7 +159,9 @@ class PagedGroupedAttention:
         H, G = self.heads, self.kv_heads
         q3 = q.unflatten(1, (H, self.dim))
         q_norm, k_norm = self.q_norm, self.k_norm
-        if self.whole_norm:
+        if self.tied_values:
+            v = k  # stored as projected; the launch below turns the keys on their way into the cache and leaves the projection as it is
+        if self.whole_norm or self.tied_values:
             # each projection as ONE row: norm, rotation (by tables that the step's layers share) and the store into the cache in one launch
             r = self.rot or {"dims": 0, "base": 1.0, "interleaved": False}
             tables = plan.rope_tables(r["dims"], r["base"], r["factor"], r["ramp"]) if r["dims"] else None
