@@ -161,7 +161,7 @@ int tlb_moe_combine_tanh(float *x, const float *pair_out, const float *gate, con
                          const void *next_b, void *h, int rows, int dim, int dtype, void *stream) {
     if (rows <= 0) return TL_OK;
     TanhNormArgs post{post_w, post_b, post_alpha}, next{next_w, next_b, next_alpha};
-    if (!x || !pair_out || !gate || top <= 0 || dim <= 0 || (idx && !h_in) || h == h_in || !norm_ok(post) || (h && !norm_ok(next)))
+    if (!x || !pair_out || !gate || top <= 0 || dim <= 0 || (idx && !h_in) || (h && h == h_in) || !norm_ok(post) || (h && !norm_ok(next)))
         return tl::fail(TL_EINVAL, "moe_combine_tanh: bad argument");
     MixArgs mix{pair_out, gate, shared_gate, shared, h_in, idx, experts, top};
     TLB_DISPATCH(dtype, "moe_combine_tanh", launch_step<T, kFromExperts>(x, nullptr, nullptr, nullptr, nullptr, 0, mix, post, next, h, rows, dim, as_stream(stream)));

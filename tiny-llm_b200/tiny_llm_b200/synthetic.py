@@ -628,3 +628,87 @@ def synthetic_zalazen(config: dict, seed: int = 0, dtype=torch.bfloat16, sharp: 
 
 
 save_zalazen = save_voluzen
+
+
+# ---- Nomudra (chunked attention whose values are its keys / matrix memory, tanh norms around every sublayer; nomudra.py) ----
+def nomudra_config(*, width=96, vocab=200, pattern="MmAmMnAm", heads=4, kv_heads=2, dim=16, chunks=(24,), rot_dims=8, rot_base=20000.0, scale=None, mem_heads=3,
+                   mem_dim=16, mem_vdim=24, gate_cap=9.0, experts=6, identity=2, top=2, groups=(2, 1), expert_ff=40, limit=1.2, shared_ff=72, shared_limit=2.0,
+                   eps=1e-5) -> dict:
+    """A config.json for a stack spelled by ``pattern``, two letters a layer: the mixer (``A`` attention, ``M`` matrix memory) and the
+    feed-forward (``m`` experts, ``n`` none).  ``chunks``: the attention layers' chunk sizes, taken in turn; ``groups`` = (count,
+    keep) or None; ``shared_ff`` 0 = no shared expert; ``rot_dims`` 0 = no rotation."""
+    if len(pattern) % 2:
+        raise ValueError("the pattern is pairs of letters: mixer, feed-forward")
+    layers, seen = [], 0
+    for mixer_letter, ff_letter in zip(pattern[0::2], pattern[1::2]):
+        if mixer_letter not in "AM" or ff_letter not in "mn":
+            raise ValueError(f"unknown layer {mixer_letter + ff_letter!r}")
+        if mixer_letter == "A":
+            mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "mask": {"size": chunks[seen % len(chunks)]},
+                     "scale": float(scale if scale is not None else dim ** -0.5)}
+            if rot_dims:
+                mixer["rot"] = {"base": rot_base, "dims": rot_dims}
+            seen += 1
+        else:
+            mixer = {"heads": mem_heads, "dim": mem_dim, "vdim": mem_vdim, "gate_cap": gate_cap}
+        mlp = None
+        if ff_letter == "m":
+            router = {"experts": experts, "identity": identity, "top": top}
+            if groups:
+                router["groups"] = {"count": groups[0], "keep": groups[1]}
+            mlp = {"kind": "moe", "expert": {"ff": expert_ff, "limit": limit}, "router": router}
+            if shared_ff:
+                mlp["shared"] = {"ff": shared_ff, "limit": shared_limit}
+        layers.append({"type": "attention" if mixer_letter == "A" else "mlstm", "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Nomudra", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": layers}
+
+
+def synthetic_nomudra(config: dict, seed: int = 0, dtype=torch.bfloat16, sharp: float = 1.0) -> dict:
+    """Random tensors for ``config`` under the checkpoint's names (CPU, seeded); ``sharp`` scales the attention layers' queries, so
+    that single keys stand out in the softmax."""
+    gen = torch.Generator().manual_seed(seed)
+    D = config["width"]
+
+    def mat(out_dim, in_dim, gain=1.0):
+        return (torch.randn(out_dim, in_dim, generator=gen) * (gain / in_dim**0.5)).to(dtype)
+
+    def vec(n, centre, spread):
+        return (centre + spread * torch.randn(n, generator=gen)).to(dtype)
+
+    tensors = {"embed": torch.randn(config["vocab"], D, generator=gen).to(dtype), "head": mat(config["vocab"], D)}
+
+    def norm(name, alpha):
+        tensors[name], tensors[name + ".b"] = vec(D, 1.0, 0.2), vec(D, 0.0, 0.1)
+        tensors[name + ".alpha"] = torch.tensor(alpha * (0.8 + 0.4 * torch.rand((), generator=gen).item())).to(dtype)
+
+    norm("embed.norm", 0.8), norm("final.norm", 0.6)
+    for i, layer in enumerate(config["layers"]):
+        m, p = layer["mixer"], f"l{i}.mix."
+        norm(f"l{i}.norm1", 0.6), norm(f"l{i}.norm1b", 1.1)
+        H, dk = m["heads"], m["dim"]
+        if layer["type"] == "attention":
+            G = m["kv_heads"]
+            tensors[p + "q"], tensors[p + "q.b"] = mat(H * dk, D, 2.0 * sharp), vec(H * dk, 0.0, 0.5)
+            tensors[p + "k"], tensors[p + "k.b"] = mat(G * dk, D, 2.0), vec(G * dk, 0.0, 0.5)
+            tensors[p + "g"], tensors[p + "o"], tensors[p + "o.b"] = mat(H * dk, D, 2.0), mat(D, H * dk), vec(D, 0.0, 0.2)
+        else:
+            dv = m["vdim"]
+            tensors[p + "q"], tensors[p + "k"], tensors[p + "v"], tensors[p + "g"] = mat(H * dk, D, 2.0), mat(H * dk, D, 2.0), mat(H * dv, D), mat(H * dv, D, 2.0)
+            tensors[p + "i"], tensors[p + "i.b"] = mat(H, D, 3.0), vec(H, -1.0, 1.0)   # now and then a token far above the rest
+            tensors[p + "f"], tensors[p + "f.b"] = mat(H, D, 2.0), vec(H, 4.0, 2.0)    # mostly near 1: a long memory
+            tensors[p + "norm"], tensors[p + "o"] = vec(H * dv, 1.0, 0.2), mat(D, H * dv)
+        mlp = layer.get("mlp")
+        if not mlp:
+            continue
+        norm(f"l{i}.norm2", 0.6), norm(f"l{i}.norm2b", 1.1)
+        r, q = mlp["router"], f"l{i}.mlp."
+        outputs = r["experts"] + r.get("identity", 0)
+        tensors[q + "router"], tensors[q + "correction"] = mat(outputs, D, 2.0), vec(outputs, -0.1, 0.1)
+        for part, ff in [(f"e{k}.", mlp["expert"]["ff"]) for k in range(r["experts"])] + ([("shared.", mlp["shared"]["ff"])] if mlp.get("shared") else []):
+            tensors[q + part + "gate"], tensors[q + part + "up"], tensors[q + part + "down"] = mat(ff, D, 2.0), mat(ff, D, 2.0), mat(D, ff)
+        if mlp.get("shared"):
+            tensors[q + "shared.sg"] = mat(1, D, 2.0)
+    return tensors
+
+
+save_nomudra = save_voluzen
