@@ -44,6 +44,9 @@ Numbers on the JSON line (decode):
   --workload zalazen  (not a BASELINE config) the Zalazen design - windowed attention with kept first positions, sinks and gates beside a
                       gated feed-forward, pair embedding - at two real-layer sizes beside Bapovik's attention layers of equal size, and its
                       kernels against their rooflines.
+  --workload nomudra  (not a BASELINE config) the Nomudra design - matrix memory and chunked attention in turn, tanh norms around every
+                      sublayer, grouped experts with a gated shared expert - at two real-layer sizes beside Senurax of equal size, and its
+                      kernels against their rooflines.
   --workload bapovik  (not a BASELINE config) the Bapovik design - windowed / chunked attention beside a recurrent mixer, experts,
             bf16 weights - at two sizes beside Voluzen of equal size, and the design's kernels alone against the measured peaks
   cpu_baseline  the reference's CPU path (oracle.model: dense bf16 weights, readable operators) on the
@@ -1835,13 +1838,216 @@ def run_zalazen(args) -> None:
                       "steps": steps, "warmup": warmup, "peaks": measured_peaks(), "clocks": clocks, "sizes": results}), flush=True)
 
 
+# ------------------------------------------------------------------ workload: nomudra (chunked attention whose values are its keys / matrix memory, grouped experts; beside Senurax of equal size)
+NOMUDRA_SIZES = {
+    # four layers at sizes that resemble real models of this kind: matrix memory and chunked attention in turn, experts in each.  The
+    # Senurax arm (the framework's closest model: fp32 stream, a decayed linear-attention layer and a softmax-attention layer in turn,
+    # gated experts with identity experts, state slots beside the paged cache, the same ragged step) has the same width, depth, heads,
+    # head sizes and experts; it has no shared expert, and its attention layers carry a delta rule of the memory's size beside the attention.
+    "w1024": dict(width=1024, vocab=32768, pattern="MmAmMmAm", heads=8, kv_heads=2, dim=128, chunks=(1024,), rot_dims=64, rot_base=100000.0, mem_heads=4, mem_dim=128,
+                  mem_vdim=256, gate_cap=15.0, experts=14, identity=2, top=2, groups=(4, 2), expert_ff=512, limit=7.0, shared_ff=512, shared_limit=7.0),
+    "w2048": dict(width=2048, vocab=32768, pattern="MmAmMmAm", heads=16, kv_heads=4, dim=128, chunks=(1024,), rot_dims=64, rot_base=100000.0, mem_heads=8, mem_dim=128,
+                  mem_vdim=256, gate_cap=15.0, experts=60, identity=4, top=6, groups=(8, 4), expert_ff=1408, limit=7.0, shared_ff=1408, shared_limit=7.0),
+}
+
+
+def _nomudra_kernels(cfg: dict, device, prompt: int, batch: int, context: int) -> dict:
+    """The kernels the design added or extended, alone at this size, CUDA-event timed after warm-up, each against the roofline
+    of its kind (measured copy bandwidth for row kernels and scans, measured cuBLAS bf16 burst for contractions), the like kernel
+    of the framework's other models beside it (``like_...``); between repetitions a 256 MB buffer is rewritten to flush L2."""
+    from extensions_b200.tiny_llm_ext_b200 import blocks
+    from tiny_llm_b200.layer_norm import TanhNorm
+
+    peaks = measured_peaks()
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=device)
+    bf = torch.bfloat16
+
+    def timed(fn, reps=7):
+        for _ in range(3):
+            fn()
+        best = []
+        for _ in range(reps):
+            flush.fill_(1)
+            best.append(cuda_time_ms(fn))
+        return statistics.median(best)
+
+    def stream(nbytes, ms, **more):
+        return dict(more, ms=round(ms, 4), gbs=round(nbytes / ms / 1e6, 1), of_measured_hbm=round(nbytes / ms / 1e6 / peaks["hbm_gbs"], 4))
+
+    def math(flops, ms, **more):
+        return dict(more, ms=round(ms, 4), tflops=round(flops / ms / 1e9, 1), of_measured_bf16_burst=round(flops / ms / 1e9 / peaks["bf16_tflops"], 4))
+
+    rnd = lambda *shape: torch.randn(shape, device=device).to(bf)
+    out = {}
+    D, V, rows = cfg["width"], cfg["vocab"], 32768
+
+    # ---- tanh norms around the stream
+    post, following = (TanhNorm(torch.ones(D, device=device).to(bf), torch.zeros(D, device=device).to(bf), torch.tensor(0.7)) for _ in range(2))
+    w1 = torch.ones(D, device=device).to(bf)
+    x, y = torch.randn((rows, D), device=device), torch.randn((rows, D), device=device)
+    for n, name in ((rows, ""), (batch, "_decode")):
+        xs, ys = x[:n], y[:n]
+        ms = timed(lambda: post.follow(xs, ys, following))
+        out["tanh_step" + name] = stream(n * D * (4 + 4 + 4 + 2), ms, rows=n)
+        ms = timed(lambda: blocks.add_norm(xs, ys, None, w1, 1e-6))
+        out["like_add_norm" + name] = stream(n * D * (4 + 4 + 4 + 2), ms, rows=n)
+    ids, table = torch.randint(0, V, (rows,), dtype=torch.int32, device=device), rnd(V, D)
+    ms = timed(lambda: post.embed(ids, table, following))
+    out["tanh_embed"] = stream(rows * D * (2 + 4 + 2), ms, rows=rows)
+    ms = timed(lambda: blocks.embed_rows(ids, table))
+    out["like_embed_rows"] = stream(rows * D * (2 + 4 + 2), ms, rows=rows)
+    del table, y
+
+    # ---- matrix memory
+    H, dk, dv, cap = cfg["mem_heads"], cfg["mem_dim"], cfg["mem_vdim"], cfg["gate_cap"]
+
+    def memory(tokens_per_seq, seqs, start, like):
+        T = tokens_per_seq * seqs
+        q, k, v = rnd(T, H, dk), rnd(T, H, dk), rnd(T, H, dv)
+        info = torch.tensor([(s * tokens_per_seq, tokens_per_seq, start, s) for s in range(seqs)], dtype=torch.int32, device=device)
+        state = torch.zeros((seqs, H, dk, dv + (not like)), device=device)
+        args = dict(q_scale=dk ** -0.5, seq_info=info, state=state, max_tokens=tokens_per_seq)
+        if like:
+            decay = torch.linspace(0.9, 0.999, H, device=device)
+            return timed(lambda: blocks.decay_scan(q, k, v, None, None, head_decay=decay, **args))
+        steps = torch.rand((T, H, 2), device=device)
+        return timed(lambda: blocks.decay_scan(q, k, v, steps, None, decay_kind=blocks.DECAY_GIVEN, normaliser=True, **args))
+
+    def gates(tokens_per_seq, seqs, start, inline):
+        T = tokens_per_seq * seqs
+        z, h, w, b = torch.randn((T, 2 * H), device=device), rnd(T, D), rnd(2 * H, D), rnd(2 * H)
+        info = torch.tensor([(s * tokens_per_seq, tokens_per_seq, start, s) for s in range(seqs)], dtype=torch.int32, device=device)
+        state = torch.zeros((seqs, H), device=device)
+        return timed(lambda: blocks.matrix_memory_gates(None if inline else z, h=h, w=w, bias=b, cap=cap, heads=H, seq_info=info, state=state, max_tokens=tokens_per_seq))
+
+    for like in (False, True):
+        name, cols = ("like_retention_scan", dv) if like else ("matrix_memory_scan", dv + 1)
+        ms = memory(prompt, 1, 0, like)
+        nbytes = prompt * H * (2 * dk * 2 + dv * 2 + cols * 4 + (0 if like else 8))
+        out[name + "_prefill"] = stream(nbytes, ms, tokens=prompt, gflops=round(4.0 * prompt * H * dk * cols / ms / 1e6, 1), note="three launches over 64-token segments; bound by instruction issue, not bytes")
+        ms = memory(1, batch, context, like)
+        out[name + "_decode"] = stream(batch * H * dk * cols * 4 * 2, ms, batch=batch)
+    out["memory_gates_prefill"] = stream(prompt * H * (8 + 8 + 4), gates(prompt, 1, 0, False), tokens=prompt, note="a scan over the prompt per head: one CTA each")
+    out["memory_gates_decode"] = stream(batch * (D * 2 + H * 12) + 2 * H * D * 2, gates(1, batch, context, True), batch=batch, note="with the two gates' projections")
+    big = 8192
+    o, gate, nw = torch.randn((big, H, dv + 1), device=device), rnd(big, H * dv), rnd(H * dv)
+    floor = torch.rand((big, H), device=device)
+    ms = timed(lambda: blocks.head_norm_gate(o, nw, 1e-6, gate, act=2, floor=floor, den_eps=1e-6))
+    out["normaliser_norm_gate"] = stream(big * H * dv * (4 + 2 + 2), ms, rows=big)
+    plain = o[:, :, :dv].contiguous()
+    ms = timed(lambda: blocks.head_norm_gate(plain, nw, 1e-6, gate, act=2))
+    out["like_head_norm_gate"] = stream(big * H * dv * (4 + 2 + 2), ms, rows=big)
+    del o, gate, plain
+
+    # ---- attention
+    AH, G, d, page, chunk, rot = cfg["heads"], cfg["kv_heads"], cfg["dim"], 64, cfg["chunks"][0], cfg["rot_dims"]
+    forms = blocks.paged_attention_flash_forms(bf, AH, G, d, d, page)
+
+    def attention(tokens_per_seq, seqs, ctx, kernel, gated):
+        pages_per, tile = -(-ctx // page), forms[kernel]
+        slab = rnd(seqs * pages_per, page, G * 2 * d)
+        table = torch.arange(seqs * pages_per, dtype=torch.int32, device=device).view(seqs, pages_per)
+        T = tokens_per_seq * seqs
+        tok = torch.cat([torch.arange(ctx - tokens_per_seq, ctx, dtype=torch.int32) for _ in range(seqs)]).to(device)
+        tiles = torch.tensor([(s * tokens_per_seq + f, min(tile, tokens_per_seq - f), s) for s in range(seqs) for f in range(0, tokens_per_seq, tile)],
+                             dtype=torch.int32, device=device)
+        q, gate = rnd(T, AH, d), rnd(T, AH * d if gated else AH)
+        return timed(lambda: blocks.paged_attention(q, slab, table, tiles, tok, kv_heads=G, dv=d, mask=blocks.MASK_CHUNK, mask_size=chunk, scale=d ** -0.5, gate=gate,
+                                                    kernel=kernel, max_context=ctx))
+
+    for name, gated in (("chunk_attention_entry_gate", True), ("like_chunk_attention_head_gate", False)):
+        seen = sum(p % chunk + 1 for p in range(prompt))
+        out[name + "_prefill"] = math(2.0 * AH * 2 * d * seen, attention(prompt, 1, prompt, "flash", gated), kernel="flash", tokens=prompt, chunk=chunk)
+        seen = (context - 1) % chunk + 1
+        out[name + "_decode"] = stream(batch * seen * G * 2 * d * 2, attention(1, batch, context, "flash_split", gated), kernel="flash_split", batch=batch, context=context)
+    pos, seq = torch.arange(rows, dtype=torch.int32, device=device), torch.zeros(rows, dtype=torch.int32, device=device)
+    wide = rnd(rows, (AH + 2 * G + AH) * d)
+    q, k, v = wide[:, : AH * d], wide[:, AH * d : (AH + G) * d], wide[:, (AH + G) * d : (AH + 2 * G) * d]
+    slab = torch.empty((rows // page, page, G * 2 * d), dtype=bf, device=device)
+    block_table = torch.arange(rows // page, dtype=torch.int32, device=device).view(1, -1)
+    angles = blocks.rope_table(pos, dims=rot, base=cfg["rot_base"])
+    qw, kw = rnd(AH * d), rnd(G * d)
+    for n, name in ((rows, ""), (batch, "_decode")):
+        args = dict(heads=AH, kv_heads=G, eps=1e-6, rot_dims=rot, base=cfg["rot_base"], tok_pos=pos[:n], tok_seq=seq[:n], block_table=block_table, slab=slab,
+                    rope=(angles[0][:n], angles[1][:n]))
+        ms = timed(lambda: blocks.qk_whole_prepare(q[:n], k[:n], k[:n], **args))
+        out["turned_keys_and_values_store" + name] = stream(n * (2 * AH * d + 3 * G * d) * 2, ms, rows=n, note="queries in place; keys read once, stored turned and as they are")
+        ms = timed(lambda: blocks.qk_whole_prepare(q[:n], k[:n], v[:n], q_norm=qw, k_norm=kw, **args))
+        out["like_whole_norm_store" + name] = stream(n * (2 * AH * d + 4 * G * d) * 2, ms, rows=n)
+    del wide, q, k, v, slab
+
+    # ---- experts
+    E, ident, top, ff, sff = cfg["experts"], cfg["identity"], cfg["top"], cfg["expert_ff"], cfg["shared_ff"]
+    wg, wu = ((torch.randn((E, ff, D), device=device) / D**0.5).to(bf) for _ in range(2))
+    wd = (torch.randn((E, D, ff), device=device) / ff**0.5).to(bf)
+    router_w, bias, side_w = rnd(E + ident, D), torch.zeros(E + ident, device=device).to(bf), rnd(1, D)
+    for n, name in ((prompt, "_prefill"), (batch, "_decode")):
+        h, shared = rnd(n, D), rnd(n, D)
+        route = lambda: blocks.moe_route(h, router_w, None, top, blocks.SCORE_SOFTMAX_ALL, bias, 1.0, cfg["groups"], side_w)
+        ms = timed(route)
+        out["grouped_route_side_gate" + name] = math(2.0 * n * (E + ident + 1) * D, ms, tokens=n)
+        ms = timed(lambda: blocks.moe_route(h, router_w, None, top, blocks.SCORE_SOFTMAX_ALL, bias, 1.0))
+        out["like_route" + name] = math(2.0 * n * (E + ident) * D, ms, tokens=n)
+        idx, gate, side = route()
+        xs = x[:n]
+        fused = timed(lambda: blocks.moe_experts(h, idx, gate, wg, wu, wd, blocks.ACT_CLAMPED_SWISH, shared, identity=True, limit=7.0, slope=1.702, shared_gate=side,
+                                                 into=(xs, post, following)))
+        like = timed(lambda: blocks.add_norm(xs, blocks.moe_experts(h, idx, gate, wg, wu, wd, blocks.ACT_SILU, shared, identity=True), None, w1, 1e-6))
+        real = float((idx < E).float().mean())
+        for label, ms in (("clamped_experts_and_tanh_step", fused), ("like_silu_experts_and_add_norm", like)):
+            if n == prompt:
+                out[label + name] = math(2.0 * 3 * n * top * real * ff * D, ms, tokens=n, share_of_choices_on_real_experts=round(real, 3))
+            else:
+                out[label + name] = stream(len(set(idx[idx < E].tolist())) * 3 * ff * D * 2, ms, batch=n, note="bytes of the experts that were chosen")
+    return out
+
+
+def run_nomudra(args) -> None:
+    """Prefill and decode throughput of the Nomudra design at NOMUDRA_SIZES beside Senurax (the framework's closest model) of
+    equal size, through the same ragged step; and the design's kernels against their rooflines.  One JSON line; random
+    weights, random prompts."""
+    from tiny_llm_b200.models import model_class
+    from tiny_llm_b200.synthetic import nomudra_config, senurax_config, synthetic_nomudra, synthetic_senurax
+
+    device = torch.device("cuda:0")
+    prompt, batch, context, steps = args.prompt_len or 2048, 16, 1024, max(args.steps or 16, 4)
+    warmup = max(args.warmup, 3)
+    sampler = ClockSampler(0)
+    sampler.start()
+    results = []
+    for name, size in NOMUDRA_SIZES.items():
+        config = nomudra_config(**size)
+        model = model_class("Nomudra").from_checkpoint(config, synthetic_nomudra(config, seed=0), device=device, dtype=torch.bfloat16)
+        entry = {"size": name, "config": dict(size), "prompt_tokens": prompt, "decode_batch": batch, "decode_context": context,
+                 "nomudra": _measure_ragged(model, size["vocab"], prompt, batch, context, steps, warmup)}
+        entry["nomudra_batch1"] = _measure_ragged(model, size["vocab"], prompt, 1, context, steps, warmup)
+        entry["kernels"] = _nomudra_kernels(size, device, prompt, batch, context)
+        del model
+        torch.cuda.empty_cache()
+        ssize = dict(width=size["width"], vocab=size["vocab"], pattern="RmPmRmPm", loop=None, heads=size["heads"], kv_heads=size["kv_heads"], dim=size["dim"],
+                     vdim=size["dim"], rot_dims=size["rot_dims"], rot_factor=1.0, rec_heads=size["mem_heads"], rec_key_heads=size["mem_heads"], rec_dim=size["mem_dim"],
+                     rec_vdim=size["mem_vdim"], ret_heads=size["mem_heads"], ret_dim=size["mem_dim"], ret_vdim=size["mem_vdim"], ret_rot_dims=size["mem_dim"],
+                     experts=size["experts"], identity=size["identity"], top=size["top"], expert_ff=size["expert_ff"], router_scale=1.0, softcap=None)
+        sconfig = senurax_config(**ssize)
+        other = model_class("Senurax").from_checkpoint(sconfig, synthetic_senurax(sconfig, seed=0), device=device, dtype=torch.bfloat16)
+        entry["senurax_equal_size"] = dict(_measure_ragged(other, size["vocab"], prompt, batch, context, steps, warmup), config=ssize)
+        entry["senurax_equal_size_batch1"] = _measure_ragged(other, size["vocab"], prompt, 1, context, steps, warmup)
+        del other
+        torch.cuda.empty_cache()
+        results.append(entry)
+    clocks = sampler.stop()
+    print(json.dumps({"workload": "nomudra", "metric": "Nomudra prefill / decode tok/s beside Senurax of equal size", "unit": UNIT, "n_gpus": 1,
+                      "dtype": "bf16 (unquantised weights in both)", "data": "synthetic (random weights, random prompts)",
+                      "steps": steps, "warmup": warmup, "peaks": measured_peaks(), "clocks": clocks, "sizes": results}), flush=True)
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=None)
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--impl", choices=["ours", "reference"], default="ours")
-    ap.add_argument("--workload", choices=sorted(METRICS) + ["voluzen", "bapovik", "senurax", "norusun", "zalazen"], default="decode")
+    ap.add_argument("--workload", choices=sorted(METRICS) + ["voluzen", "bapovik", "senurax", "norusun", "zalazen", "nomudra"], default="decode")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-extra", action="store_true", help="skip the sweeps / secondary measurements under `extra`")
     ap.add_argument("--requests", type=int, default=0, help="serve/serve8k: total requests over all ranks")
@@ -1861,6 +2067,8 @@ def main() -> None:
         run_norusun(args)
     elif args.workload == "zalazen":
         run_zalazen(args)
+    elif args.workload == "nomudra":
+        run_nomudra(args)
     elif args.impl == "reference":
         run_reference(args)
     elif args.workload == "decode":

@@ -22,34 +22,97 @@ __device__ __forceinline__ int moe_src_row(int pair, int sorted_row, int top, in
     return gather == kGatherSorted ? sorted_row : gather == kGatherToken ? pair / top : pair;
 }
 
+// W consecutive entries of a row as floats.
+template <int W>
+__device__ __forceinline__ void moe_load(const float *p, float (&x)[W]) {
+    if constexpr (W == 1) x[0] = p[0];
+    else {
+        const float4 v = load4(p);
+        x[0] = v.x, x[1] = v.y, x[2] = v.z, x[3] = v.w;
+    }
+}
+template <int W>
+__device__ __forceinline__ void moe_load(const bf16 *p, float (&x)[W]) {
+    if constexpr (W == 1) x[0] = to_f(p[0]);
+    else {
+        const uint4 u = *reinterpret_cast<const uint4 *>(p);
+        const uint32_t c[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float2 f = tl::unpack2<bf16>(c[i]);
+            x[2 * i] = f.x, x[2 * i + 1] = f.y;
+        }
+    }
+}
+
+// A CTA routes TOK tokens, so that a row of weights is fetched once for all of them: their rows of h are staged in shared memory,
+// the warps share the experts, four rows of weights in flight each (a logit is one warp's dot product in a lane order fixed by the
+// width, whatever TOK and the launch are), then warp i picks token i's top-k.  W: entries per access (16 bytes where rows allow).
 // aux_w: one more row of weights that is no router output; aux[t] = sigmoid(aux_w . h_t) (the gate of a shared expert).
-// One CTA per token: the row of h is staged in shared memory as fp32, the warps share the experts (each logit is one
-// warp's dot product in a fixed lane order, so it does not depend on the launch), then warp 0 picks the top-k.
-template <typename T>
-__global__ void __launch_bounds__(256)
+template <typename T, int TOK, int W>
+__global__ void __launch_bounds__(TOK == 1 ? 1024 : 256)
 moe_route_kernel(const T *__restrict__ h, const T *__restrict__ w, const T *__restrict__ b, int tokens, int dim, int experts, int top, int scoring,
                  const T *__restrict__ choice_bias, float weight_scale, int group_count, int group_keep, const T *__restrict__ aux_w,
                  float *__restrict__ aux, int32_t *__restrict__ idx, float *__restrict__ gate) {
-    extern __shared__ float route_smem[];
-    float *x = route_smem;        // [dim]
-    float *z = route_smem + dim;  // [experts]: what the choice is made by
-    float *p_all = z + experts;   // [experts]: scoring 2, the softmax over all outputs
-    float *best = p_all + experts;  // [group_count]: the largest choice score of every group
-    const int t = blockIdx.x;
+    extern __shared__ __align__(16) unsigned char route_smem[];
+    T *x = reinterpret_cast<T *>(route_smem);  // [TOK][dim]
+    float *logits = reinterpret_cast<float *>(route_smem + (((size_t)TOK * dim * sizeof(T) + 15) & ~(size_t)15));
+    const int per_token = 2 * experts + group_count;  // [TOK][..]: see below
+    const int t0 = blockIdx.x * TOK, here = min(TOK, tokens - t0);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
-    for (int d = threadIdx.x; d < dim; d += blockDim.x) x[d] = to_f(h[(size_t)t * dim + d]);
-    __syncthreads();
-    for (int e = warp; e < experts + (aux_w ? 1 : 0); e += warps) {
-        const T *row = e < experts ? w + (size_t)e * dim : aux_w;
-        float s = 0.f;
-        for (int d = lane; d < dim; d += 32) s = fmaf(x[d], to_f(row[d]), s);
-        s = warp_sum(s);
-        if (lane != 0) continue;
-        if (e < experts) z[e] = s + (b ? to_f(b[e]) : 0.f);
-        else aux[t] = sigmoid(s);
+    for (int d = threadIdx.x * W; d < here * dim; d += blockDim.x * W) {
+        if constexpr (W == 1) x[d] = h[(size_t)t0 * dim + d];
+        else *reinterpret_cast<uint4 *>(x + d) = *reinterpret_cast<const uint4 *>(h + (size_t)t0 * dim + d);
     }
     __syncthreads();
-    if (warp != 0) return;
+    constexpr int ROWS = 4;
+    const int outputs = experts + (aux_w ? 1 : 0);
+    for (int e0 = warp; e0 < outputs; e0 += warps * ROWS) {
+        float acc[ROWS][TOK];
+        const T *row[ROWS];
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) {
+            const int e = e0 + r * warps;
+            row[r] = e < experts ? w + (size_t)e * dim : aux_w;  // past the last one: not read
+#pragma unroll
+            for (int i = 0; i < TOK; ++i) acc[r][i] = 0.f;
+        }
+        for (int d = lane * W; d < dim; d += 32 * W) {
+            float wv[ROWS][W];
+#pragma unroll
+            for (int r = 0; r < ROWS; ++r)
+                if (e0 + r * warps < outputs) moe_load<W>(row[r] + d, wv[r]);
+#pragma unroll
+            for (int i = 0; i < TOK; ++i) {
+                float xv[W];
+                moe_load<W>(x + (size_t)i * dim + d, xv);
+#pragma unroll
+                for (int r = 0; r < ROWS; ++r)
+                    if (e0 + r * warps < outputs) {
+#pragma unroll
+                        for (int j = 0; j < W; ++j) acc[r][i] = fmaf(xv[j], wv[r][j], acc[r][i]);
+                    }
+            }
+        }
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) {
+            const int e = e0 + r * warps;
+            if (e >= outputs) continue;
+#pragma unroll
+            for (int i = 0; i < TOK; ++i) {
+                const float s = warp_sum(acc[r][i]);
+                if (lane != 0 || i >= here) continue;
+                if (e < experts) logits[i * per_token + e] = s + (b ? to_f(b[e]) : 0.f);
+                else aux[t0 + i] = sigmoid(s);
+            }
+        }
+    }
+    __syncthreads();
+    if (warp >= here) return;
+    const int t = t0 + warp;
+    float *z = logits + warp * per_token;  // [experts]: what the choice is made by
+    float *p_all = z + experts;            // [experts]: scoring 2, the softmax over all outputs
+    float *best = p_all + experts;         // [group_count]: the largest choice score of every group
     if (scoring == 2) {  // scores = softmax over ALL outputs; the choice adds a bias to them, the weights do not
         float m = -INFINITY, sum = 0.f;
         for (int e = lane; e < experts; e += 32) m = fmaxf(m, z[e]);
@@ -384,12 +447,21 @@ int tlb_moe_route(const void *h, const void *w, const void *b, int tokens, int d
     if ((aux_w == nullptr) != (aux == nullptr) || group_count < 0 || group_keep < 0 || group_keep > group_count ||
         (group_count > 0 && (experts % group_count || group_keep * (experts / group_count) < top)))
         return tl::fail(TL_EINVAL, "moe_route: bad groups or side output");
-    size_t smem = ((size_t)dim + 2 * (size_t)experts + group_count) * sizeof(float);
-    if (smem > 48 * 1024) return tl::fail(TL_EINVAL, "moe_route: width %d + %d experts do not fit", dim, experts);
+    const size_t es = dtype == TL_BF16 ? 2 : 4;
+    const auto bytes = [&](int tok) { return (((size_t)tok * dim * es + 15) & ~(size_t)15) + (size_t)tok * (2 * (size_t)experts + group_count) * sizeof(float); };
+    if (bytes(1) > 48 * 1024) return tl::fail(TL_EINVAL, "moe_route: width %d + %d experts do not fit", dim, experts);
+    const bool wide = dim * es % 16 == 0 && tl::aligned16(h) && tl::aligned16(w) && (!aux_w || tl::aligned16(aux_w));
+    // four tokens a CTA once that fills the GPU; few tokens: more warps each, so that no warp walks many rows of weights
+    const bool many = tokens >= 4 * 148 * 2 && bytes(4) <= 48 * 1024;
+    const int threads = many || tokens > 148 ? 256 : 1024;
+#define TLB_ROUTE(TOK, WV)                                                                                                                         \
+    moe_route_kernel<T, TOK, WV><<<ceil_div(tokens, TOK), threads, bytes(TOK), as_stream(stream)>>>(                                                \
+        (const T *)h, (const T *)w, (const T *)b, tokens, dim, experts, top, scoring, (const T *)choice_bias, weight_scale, group_count, group_keep, \
+        (const T *)aux_w, aux, idx, gate)
     TLB_DISPATCH(dtype, "moe_route",
-                 moe_route_kernel<T><<<tokens, 256, smem, as_stream(stream)>>>((const T *)h, (const T *)w, (const T *)b, tokens, dim, experts, top, scoring,
-                                                                             (const T *)choice_bias, weight_scale, group_count, group_keep, (const T *)aux_w, aux,
-                                                                             idx, gate));
+                 if (wide) { if (many) TLB_ROUTE(4, (16 / (int)sizeof(T))); else TLB_ROUTE(1, (16 / (int)sizeof(T))); }
+                 else { if (many) TLB_ROUTE(4, 1); else TLB_ROUTE(1, 1); });
+#undef TLB_ROUTE
     TL_LAUNCH_CHECK("moe_route");
     return TL_OK;
 }
