@@ -232,3 +232,17 @@ def test_nothing_is_collected_while_a_graph_is_captured(monkeypatch):
         assert not gc.isenabled()
     finally:
         gc.enable()
+
+
+def test_a_public_function_outlives_the_import_of_the_module_of_its_name():
+    import os
+    import subprocess
+    import sys
+
+    code = ("import tiny_llm_b200, tiny_llm_b200.nomudra, tiny_llm_b200.zalazen\n"
+            "from tiny_llm_b200.paged_attention import PagedGroupedAttention\n"
+            "from tiny_llm_b200 import paged_attention\n"
+            "assert callable(paged_attention) and paged_attention.__module__ == 'tiny_llm_b200.attention'\n")
+    env = dict(os.environ, PYTHONPATH=str(Path(__file__).resolve().parent.parent / "tiny-llm_b200"))
+    run = subprocess.run([sys.executable, "-c", code], capture_output=True, text=True, env=env)
+    assert run.returncode == 0, run.stderr

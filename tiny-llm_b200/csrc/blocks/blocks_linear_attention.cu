@@ -50,7 +50,9 @@ __device__ __forceinline__ bool la_segment(int p0, int n, int c, int &lo, int &h
 // no value: v is 1 there, so that column v_cols carries the decayed sum of the keys themselves (a normaliser).  q and k may have fewer heads than v (qk_heads; head h
 // reads query/key head h / (heads / qk_heads)).  skip [heads]: o_t += skip[h] v_t.  BONUS: the read-out comes BEFORE the
 // update and sees the token's own k v^T weighted by bonus [heads, dk] instead: o_t = (S + diag(bonus) k_t v_t^T)^T q_t.
-template <typename T, int KR /* rows per lane: dk <= 4 * KR */, int kLaTokens /* tokens staged at a time */, bool BONUS>
+// SCALAR: the decay is one number per head and token (head_decay, decay_kind 3 and 4): it is read once per token, and a row of the
+// state reads 8 bytes of its token's staged numbers instead of 16.
+template <typename T, int KR /* rows per lane: dk <= 4 * KR */, int kLaTokens /* tokens staged at a time */, bool BONUS, bool SCALAR>
 __global__ void __launch_bounds__(kLaCols * kLaLanes)
 decay_scan_kernel(const T *__restrict__ q, long long q_token, long long q_head, const T *__restrict__ k, long long k_token, long long k_head,
                   const T *__restrict__ v, long long v_token, long long v_head, const float *__restrict__ z, long long z_token,
@@ -60,10 +62,11 @@ decay_scan_kernel(const T *__restrict__ q, long long q_token, long long q_head, 
                   float *__restrict__ state, long long slot_stride, int num_slots, float *__restrict__ out, int pass, int max_segments,
                   float *__restrict__ seg_state, float *__restrict__ seg_decay, int decay_kind, const T *__restrict__ a_log,
                   const T *__restrict__ bonus, int qk_heads, const T *__restrict__ skip, int v_cols) {
-    __shared__ float4 sx[kLaTokens * 4 * KR];  // per token and key channel: (decay, k, scaled q, -), one 16-byte read per row
+    __shared__ float4 sx[SCALAR ? 1 : kLaTokens * 4 * KR];   // per token and key channel: (decay, k, scaled q, k times the bonus), one 16-byte read per row
+    __shared__ float2 skq[SCALAR ? kLaTokens * 4 * KR : 1];  // SCALAR: (k, scaled q)
     __shared__ float sv[kLaTokens * kLaCols];
     __shared__ float sprod[4 * KR];
-    __shared__ float2 s_step[kLaTokens];  // decay_kind 3, 4: the token's (decay, key factor), worked out or read once per token
+    __shared__ float2 s_step[kLaTokens];  // SCALAR: the token's (decay, key factor), worked out or read once per token
     __shared__ float2 s_chan[4 * KR];     // per key channel of this head: (the decay logit's bias, the bonus), read once
     const int colblocks = (dv + kLaCols - 1) / kLaCols;
     const int s = blockIdx.x, head = blockIdx.y / colblocks, col0 = (blockIdx.y % colblocks) * kLaCols, c = blockIdx.z;
@@ -99,24 +102,25 @@ decay_scan_kernel(const T *__restrict__ q, long long q_token, long long q_head, 
     for (int t0 = 0; t0 < count; t0 += kLaTokens) {
         const int n = min(kLaTokens, count - t0);
         __syncthreads();
-        if (decay_kind == 3) {
+        if (SCALAR && decay_kind == 3) {
             if (threadIdx.x < n) {
                 const float zz = z[(size_t)(first + t0 + threadIdx.x) * z_token + head] + (z_bias ? to_f(z_bias[head]) : 0.f);
                 const float dt = zz > 20.f ? zz : log1pf(expf(zz));
                 s_step[threadIdx.x] = make_float2(expf(-rate * dt), dt);
             }
             __syncthreads();
-        } else if (decay_kind == 4) {
-            if (threadIdx.x < n) s_step[threadIdx.x] = *reinterpret_cast<const float2 *>(z + (size_t)(first + t0 + threadIdx.x) * z_token + 2 * head);
+        } else if (SCALAR) {
+            if (threadIdx.x < n)
+                s_step[threadIdx.x] = decay_kind == 4 ? *reinterpret_cast<const float2 *>(z + (size_t)(first + t0 + threadIdx.x) * z_token + 2 * head)
+                                                      : make_float2(head_decay[head], 1.f);
             __syncthreads();
         }
         for (int e = threadIdx.x; e < n * dk; e += blockDim.x) {
             int j = e / dk, d = e - j * dk;
             size_t tok = (size_t)(first + t0 + j);
             float alpha, kmul = 1.f;
-            if (head_decay) alpha = head_decay[head];
+            if (SCALAR) alpha = 0.f, kmul = s_step[j].y;
             else if (decay_kind == 2) alpha = expf(-expf(z[tok * z_token + (size_t)head * dk + d] + s_chan[d].x));
-            else if (decay_kind >= 3) alpha = s_step[j].x, kmul = s_step[j].y;
             else alpha = expf(log_sigmoid(z[tok * z_token + (size_t)head * dk + d] + s_chan[d].x) * inv_tau);
             const T *kp = k + tok * k_token + (size_t)qk_head * k_head, *qp = q + tok * q_token + (size_t)qk_head * q_head;
             float kd = to_f(kp[d]), qd = to_f(qp[d]);
@@ -130,7 +134,8 @@ decay_scan_kernel(const T *__restrict__ q, long long q_token, long long q_head, 
                 qd = qd * c + to_f(qp[other]) * sn;
             }
             kd *= kmul;
-            sx[j * 4 * KR + d] = make_float4(alpha, kd, qd * q_scale, BONUS ? kd * s_chan[d].y : 0.f);
+            if (SCALAR) skq[j * 4 * KR + d] = make_float2(kd, qd * q_scale);
+            else sx[j * 4 * KR + d] = make_float4(alpha, kd, qd * q_scale, BONUS ? kd * s_chan[d].y : 0.f);
         }
         for (int e = threadIdx.x; e < n * kLaCols; e += blockDim.x) {
             int j = e / kLaCols, d = e - j * kLaCols;
@@ -140,25 +145,32 @@ decay_scan_kernel(const T *__restrict__ q, long long q_token, long long q_head, 
         if (pass == 1) {  // the segment's decay product per key channel, in token order
             for (int d = threadIdx.x; d < dk; d += blockDim.x) {
                 float p = sprod[d];
-                for (int j = 0; j < n; ++j) p *= sx[j * 4 * KR + d].x;
+                for (int j = 0; j < n; ++j) p *= SCALAR ? s_step[j].x : sx[j * 4 * KR + d].x;
                 sprod[d] = p;
             }
         }
         for (int j = 0; j < n; ++j) {
             const float vj = sv[j * kLaCols + cidx];
-            const float4 *xa = sx + j * 4 * KR;
+            const float4 *xa = sx + (SCALAR ? 0 : j * 4 * KR);
+            const float2 *ya = skq + (SCALAR ? j * 4 * KR : 0);
+            const float keep = SCALAR ? s_step[j].x : 0.f;
+            auto staged = [&](int row) {
+                if (!SCALAR) return xa[row];
+                const float2 y = ya[row];
+                return make_float4(keep, y.x, y.y, 0.f);
+            };
             float o0 = 0.f, o1 = 0.f;
 #pragma unroll
             for (int i = 0; i < KR; i += 2) {
                 int row = r + kLaLanes * i;
                 if (row < dk) {
-                    float4 x = xa[row];
+                    float4 x = staged(row);
                     if (BONUS) o0 = fmaf(x.z, fmaf(x.w, vj, S[i]), o0);
                     S[i] = fmaf(x.x, S[i], x.y * vj);
                     if (!BONUS) o0 = fmaf(x.z, S[i], o0);
                 }
                 if (row + kLaLanes < dk) {
-                    float4 x = xa[row + kLaLanes];
+                    float4 x = staged(row + kLaLanes);
                     if (BONUS) o1 = fmaf(x.z, fmaf(x.w, vj, S[i + 1]), o1);
                     S[i + 1] = fmaf(x.x, S[i + 1], x.y * vj);
                     if (!BONUS) o1 = fmaf(x.z, S[i + 1], o1);
@@ -305,15 +317,17 @@ int tlb_decay_scan(const void *q, long long q_token, long long q_head, const voi
         seg_state = (float *)workspace;
         seg_decay = seg_state + (size_t)num_seqs * max_segments * heads * dk * dv;
     }
+    const bool scalar = head_decay || decay_kind >= 3;
+    if (scalar && bonus) return tl::fail(TL_EINVAL, "decay_scan: a bonus goes with a decay per key channel");
     const int colblocks = ceil_div(dv, kLaCols);
     cudaStream_t st = as_stream(stream);
     int kr = ceil_div(dk, kLaLanes);
-#define TLB_DS_B(KRV, PASS, GZ, BON)                                                                                                                \
-    decay_scan_kernel<T, KRV, (KRV > 32 ? 8 : 16), BON><<<dim3(num_seqs, heads * colblocks, GZ), kLaCols * kLaLanes, 0, st>>>(                                           \
+#define TLB_DS_B(KRV, PASS, GZ, BON, SCA)                                                                                                                \
+    decay_scan_kernel<T, KRV, (KRV > 32 ? 8 : 16), BON, SCA><<<dim3(num_seqs, heads * colblocks, GZ), kLaCols * kLaLanes, 0, st>>>(                                           \
         (const T *)q, q_token, q_head, (const T *)k, k_token, k_head, (const T *)v, v_token, v_head, z, z_token, (const T *)z_bias, z ? 1.0f / tau : 0.f, head_decay, \
         rope_cos, rope_sin, rope_dims, rope_interleaved, q_scale, heads, dk, dv, seq_info, state, slot_stride, num_slots, out, PASS, max_segments, seg_state, seg_decay, \
         decay_kind, (const T *)a_log, (const T *)bonus, qk_heads, (const T *)skip, v_cols)
-#define TLB_DS_K(KRV, PASS, GZ) do { if (bonus) TLB_DS_B(KRV, PASS, GZ, true); else TLB_DS_B(KRV, PASS, GZ, false); } while (0)
+#define TLB_DS_K(KRV, PASS, GZ) do { if (bonus) TLB_DS_B(KRV, PASS, GZ, true, false); else if (scalar) TLB_DS_B(KRV, PASS, GZ, false, true); else TLB_DS_B(KRV, PASS, GZ, false, false); } while (0)
 #define TLB_DS(PASS, GZ) TLB_DISPATCH(dtype, "decay_scan", if (kr <= 8) TLB_DS_K(8, PASS, GZ); else if (kr <= 16) TLB_DS_K(16, PASS, GZ); else if (kr <= 32) TLB_DS_K(32, PASS, GZ); else TLB_DS_K(64, PASS, GZ))
     if (!segmented) {
         TLB_DS(0, 1);

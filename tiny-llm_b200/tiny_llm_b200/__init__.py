@@ -2,6 +2,8 @@
 re-hosted on torch tensors over the sm_100a extension.  The public names are
 those of ``tiny_llm_ref`` (``/root/reference/src/tiny_llm_ref/__init__.py``)."""
 
+# The module and a public function share a name.  The module is loaded first, so that no later import of it rebinds the name.
+from . import paged_attention as _paged_attention_module  # noqa: F401
 from .attention import *  # noqa: F401,F403
 from .attention import paged_attention, scaled_dot_product_attention_grouped, scaled_dot_product_attention_simple, causal_mask
 from .basics import linear, silu, softmax
