@@ -53,7 +53,7 @@ __device__ __forceinline__ bool la_segment(int p0, int n, int c, int &lo, int &h
 // SCALAR: the decay is one number per head and token (head_decay, decay_kind 3 and 4): it is read once per token, and a row of the
 // state reads 8 bytes of its token's staged numbers instead of 16.
 template <typename T, int KR /* rows per lane: dk <= 4 * KR */, int kLaTokens /* tokens staged at a time */, bool BONUS, bool SCALAR>
-__global__ void __launch_bounds__(kLaCols * kLaLanes)
+__global__ void __launch_bounds__(kLaCols * kLaLanes, SCALAR && KR == 32 ? 8 : 1)
 decay_scan_kernel(const T *__restrict__ q, long long q_token, long long q_head, const T *__restrict__ k, long long k_token, long long k_head,
                   const T *__restrict__ v, long long v_token, long long v_head, const float *__restrict__ z, long long z_token,
                   const T *__restrict__ z_bias, float inv_tau, const float *__restrict__ head_decay, const float *__restrict__ rope_cos,
