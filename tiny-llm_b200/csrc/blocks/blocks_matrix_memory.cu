@@ -28,7 +28,7 @@ matrix_memory_gates_kernel(const float *__restrict__ z, long long z_token, const
     float *mine = state + (size_t)(slot_ok ? slot : 0) * slot_stride + head;
     const float bi = bias ? to_f(bias[head]) : 0.f, bf = bias ? to_f(bias[heads + head]) : 0.f;
     float carry = start > 0 && slot_ok ? *mine : 0.f;
-    const int batch = z ? (int)blockDim.x : 1;  // tokens per round
+    const int batch = z ? (int)blockDim.x : 1;  // tokens at a time
     for (int t0 = 0; t0 < count; t0 += batch) {
         const int t = t0 + (int)threadIdx.x;
         const bool live = z ? t < count : threadIdx.x == 0;
